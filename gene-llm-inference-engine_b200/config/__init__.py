@@ -4,9 +4,10 @@ from .nipadra import NipadraConfig
 from .gekupel import GekupelConfig
 from .pinorax import PinoraxConfig
 from .fovezen import FovezenConfig
+from .mimolix import MimolixConfig
 from .registry import (Architecture, known_architectures, parse_config, register_architecture,
                        resolve_architecture)
 
-__all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "LlamaConfig", "NipadraConfig", "GekupelConfig", "PinoraxConfig", "FovezenConfig",
+__all__ = ["ConfigError", "LayerSpec", "ModelSpec", "PartSpec", "ScheduleEntry", "LlamaConfig", "NipadraConfig", "GekupelConfig", "PinoraxConfig", "FovezenConfig", "MimolixConfig",
            "RopeScaling", "parse_rope_scaling", "Architecture", "known_architectures", "parse_config",
            "register_architecture", "resolve_architecture"]

@@ -50,10 +50,12 @@ class LayerSpec:
 class ScheduleEntry:
     """One run of a layer. ``cache_of`` names the layer whose cache (pages or state) this run
     reads and writes; ``None`` means the layer's own. ``writes_cache`` False makes the run a
-    reader only (the keys and values of the owner are used as they are)."""
+    reader only (the keys and values of the owner are used as they are). ``stream_input``: the residual stream is
+    replaced by the model's ``stream_input`` part right before this run."""
     layer: int
     cache_of: Optional[int] = None
     writes_cache: bool = True
+    stream_input: bool = False
 
 
 @dataclass
@@ -69,6 +71,9 @@ class ModelSpec:
     embedding_scale: float = 1.0   # multiplier on embedding rows (1 = none)
     # what is added to the embedding's output per position (kind "learned": a table of vectors); None = nothing
     embedding_position: Optional[PartSpec] = None
+    # what replaces the stream ahead of the runs whose schedule entry says so (kind "embedding_mix": a product over the
+    # stream and the embedding's output); None = nothing
+    stream_input: Optional[PartSpec] = None
     logit_transform: Optional[PartSpec] = None   # applied to the logits after the head (a scale, a soft cap); None = none
     # a design without a context length of its own: ``max_position`` is then only the engine's default, and the
     # caller's limit may exceed it
@@ -91,3 +96,5 @@ class ModelSpec:
                 raise ConfigError(f"schedule names layer {e.layer}, the model has {n}")
             if e.cache_of is not None and not (0 <= e.cache_of < n):
                 raise ConfigError(f"schedule entry reads the cache of layer {e.cache_of}, the model has {n}")
+            if e.stream_input and self.stream_input is None:
+                raise ConfigError(f"schedule replaces the stream ahead of layer {e.layer}, but the model has no part for it")

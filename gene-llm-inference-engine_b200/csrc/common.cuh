@@ -120,6 +120,13 @@ __device__ __forceinline__ float gated_value(float g, float u, int act, float li
     return g * (1.0f / (1.0f + expf(-g))) * u;
 }
 
+// What an ungated feed-forward applies to its first product, 32-bit: 0 nothing, 1 the square of ReLU.
+enum PlainAct : int { kPlainNone = 0, kPlainRelu2 = 1, kPlainCount = 2 };
+__device__ __forceinline__ float plain_value(float z, int act) {
+    if (act == kPlainRelu2) { z = fmaxf(z, 0.f); return z * z; }
+    return z;
+}
+
 template <typename... KArgs, typename... Args>
 inline void launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args&&... args) {
     cudaLaunchConfig_t cfg = {};

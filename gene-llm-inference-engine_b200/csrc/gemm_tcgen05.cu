@@ -221,6 +221,7 @@ struct RopeStoreParams {
 struct TcParams {
     void* C;
     int c_bf16;              // 0: C is float, 1: C is bfloat16
+    int plain_act;           // bfloat16 C: a PlainAct code applied to the sum before it is rounded
     int accumulate;          // C += product (float C only)
     int rows_p, rows_q, K;
     long long stride_p, stride_q;   // C[p * stride_p + q * stride_q]
@@ -253,7 +254,7 @@ __device__ __forceinline__ void store_row_chunk(const TcParams& p, bool c_bf16, 
         __nv_bfloat16* c = static_cast<__nv_bfloat16*>(p.C) + base;
 #pragma unroll
         for (int j = 0; j < 16; ++j)
-            if (j < n) c[j * p.stride_q] = __float2bfloat16_rn(v[j]);
+            if (j < n) c[j * p.stride_q] = __float2bfloat16_rn(plain_value(v[j], p.plain_act));
     } else if (accumulate) {
         // all loads first, then all stores: the sixteen read-modify-writes overlap instead of
         // waiting for one another
@@ -839,7 +840,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
 // Epilogues: store 32-bit, add to 32-bit, or SwiGLU: the tile's first half of columns are gate
 // channels and the second half the matching up channels (two TMA loads per stage from the
 // [gate; up] weight), and silu(gate) * up is stored as bfloat16.
-enum TcEpilogue : int { kEpiStoreF32 = 0, kEpiAddF32 = 1, kEpiSwiGLU = 2, kEpiRopeStore = 3 };
+// kEpiActBF16: act(sum) rounded to bfloat16, the first product of an ungated feed-forward.
+enum TcEpilogue : int { kEpiStoreF32 = 0, kEpiAddF32 = 1, kEpiSwiGLU = 2, kEpiRopeStore = 3, kEpiActBF16 = 4 };
 
 __device__ __forceinline__ void mbar_arrive(uint32_t bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
@@ -927,7 +929,7 @@ struct TcPersistentParams {
     int rows_p, rows_q, K;       // tokens, output columns of the accumulator tile space, reduction length
     int tiles_p, tiles_q;
     int up_row_offset;           // SwiGLU: row of the first up channel in the weight (= I)
-    int gate_act;                // SwiGLU epilogue: what is applied to the gate (a GateAct code)
+    int gate_act;                // SwiGLU epilogue: what is applied to the gate (a GateAct code); kEpiActBF16: a PlainAct code
     float act_limit;             //   its limit (capped swish)
     const float* gate_up_bias;   //   optional: a bias on the gate channels and, up_row_offset values further, on the up channels
     int bias_vec;                //   both halves of the bias start on 16-byte boundaries: whole groups of 8 channels take 16-byte loads
@@ -1227,7 +1229,8 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
                 }
                 continue;
             }
-            constexpr int kChunks = (EPI == kEpiSwiGLU) ? BLOCK_Q / 128 : BLOCK_Q / 32;   // TMA stores per tile
+            // TMA stores per tile
+            constexpr int kChunks = (EPI == kEpiSwiGLU) ? BLOCK_Q / 128 : (EPI == kEpiActBF16) ? BLOCK_Q / 64 : BLOCK_Q / 32;
             if (group >= kChunks) {                               // a tile with a single chunk: this group has nothing to read
                 tc_fence_before();
                 acc_empty_arrive(buf);
@@ -1285,6 +1288,27 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
                                 make_uint4(packed[0], packed[1], packed[2], packed[3]);
                         }
                     }
+                } else if (EPI == kEpiActBF16) {
+                    // 64 output channels per store, in two halves of 32
+#pragma unroll
+                    for (int half = 0; half < 2; ++half) {
+                        tmem_ld_x16(tmem_d + c * 64 + half * 32, r);
+                        tmem_ld_x16(tmem_d + c * 64 + half * 32 + 16, r + 16);
+                        tmem_ld_wait();
+                        if (last && half == 1) { tc_fence_before(); acc_empty_arrive(buf); }
+#pragma unroll
+                        for (int q4 = 0; q4 < 4; ++q4) {          // 8 channels = 16 bytes of bfloat16 per step
+                            uint32_t packed[4];
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const __nv_bfloat162 hb = __floats2bfloat162_rn(plain_value(__uint_as_float(r[q4 * 8 + 2 * e]), p.gate_act),
+                                                                                plain_value(__uint_as_float(r[q4 * 8 + 2 * e + 1]), p.gate_act));
+                                packed[e] = *reinterpret_cast<const uint32_t*>(&hb);
+                            }
+                            *reinterpret_cast<uint4*>(stg + row * 128 + (((half * 4 + q4) ^ (row & 7)) * 16)) =
+                                make_uint4(packed[0], packed[1], packed[2], packed[3]);
+                        }
+                    }
                 } else {
                     tmem_ld_x16(tmem_d + c * 32, r);
                     tmem_ld_x16(tmem_d + c * 32 + 16, r + 16);
@@ -1298,7 +1322,8 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_p, const __gri
                 fence_async_smem();
                 group_sync();
                 if (leader) {
-                    const int col = (EPI == kEpiSwiGLU) ? tile_q * (BLOCK_Q / 2) + c * 64 : tile_q * BLOCK_Q + c * 32;
+                    const int col = (EPI == kEpiSwiGLU) ? tile_q * (BLOCK_Q / 2) + c * 64
+                                    : tile_q * BLOCK_Q + c * (EPI == kEpiActBF16 ? 64 : 32);
                     if (EPI == kEpiAddF32) tma_reduce_add_2d(&map_c, smem_u32(stg), col, out_row);
                     else tma_store_2d(&map_c, smem_u32(stg), col, out_row);
                     bulk_commit();
@@ -1598,7 +1623,11 @@ static int run_gemm_tc(const void* A, const void* W, void* C, int c_dtype, int a
                "gemm_tc: K=%d and the row strides (%lld, %lld) must be multiples of 8 (16-byte rows for TMA)", K, lda, ldw);
     GI_REQUIRE((reinterpret_cast<uintptr_t>(A) % 16 == 0) && (reinterpret_cast<uintptr_t>(W) % 16 == 0),
                "gemm_tc: operands must be 16-byte aligned");
+    const int plain_act = c_dtype >> 8;                     // (the code's upper bits: an activation of the output)
+    c_dtype &= 0xff;
     GI_REQUIRE(c_dtype == kF32 || c_dtype == kBF16, "gemm_tc: unsupported output dtype code %d", c_dtype);
+    GI_REQUIRE(plain_act >= 0 && plain_act < kPlainCount && (plain_act == 0 || c_dtype == kBF16),
+               "gemm_tc: an activation (code %d) goes with a bfloat16 output", plain_act);
     GI_REQUIRE(!(accumulate && c_dtype != kF32), "gemm_tc: accumulation needs a 32-bit output");
     GI_REQUIRE(block_q == 16 || block_q == 32 || block_q == 64 || block_q == 128 || block_q == 256,
                "gemm_tc: block_q=%d is not one of 16, 32, 64, 128, 256", block_q);
@@ -1613,6 +1642,7 @@ static int run_gemm_tc(const void* A, const void* W, void* C, int c_dtype, int a
     }
     p.C = C;
     p.c_bf16 = c_dtype == kBF16;
+    p.plain_act = plain_act;
     p.accumulate = accumulate;
     p.K = K;
     p.splits = splits;
@@ -1727,7 +1757,7 @@ __global__ void reduce_splits_kernel(const float* __restrict__ ws, float* __rest
 
 // Many tokens, one persistent CTA per SM. epilogue 0: C[M,N] = A W^T (32-bit); 1: C += A W^T (32-bit);
 // 2: W is [2N, K] = [gate; up] and C[M,N] = act(A Wgate^T) * (A Wup^T) as bfloat16, act named by the bits above the
-// epilogue's low byte (0 SiLU, 1 ReLU, 2 tanh-GELU).
+// epilogue's low byte (0 SiLU, 1 ReLU, 2 tanh-GELU); 4: C[M,N] = act(A W^T) as bfloat16, act a PlainAct code there.
 // block_q: 256 or 128 accumulator columns per tile.
 // splits > 1 (epilogues 0 and 1, N a multiple of 4, at most 8): K is cut into ranges whose tiles are work
 // items of their own; their results go to `workspace` (splits x ceil(M / 128) x 128 x N floats) and a
@@ -1743,10 +1773,12 @@ static int gi_gemm_tc_persistent_impl(const void* A, const void* W, void* C, int
                "gemm_tc: K=%d and the row strides (%lld, %lld) must be multiples of 8 (16-byte rows for TMA)", K, lda, ldw);
     const int gate_act = epilogue >> 8;
     epilogue &= 0xff;
-    GI_REQUIRE(epilogue >= 0 && epilogue <= 2 && gate_act >= 0 && gate_act < kActCount && (gate_act == 0 || epilogue == kEpiSwiGLU),
+    GI_REQUIRE(((epilogue >= 0 && epilogue <= 2) || epilogue == kEpiActBF16) && gate_act >= 0 &&
+               gate_act < (epilogue == kEpiActBF16 ? static_cast<int>(kPlainCount) : static_cast<int>(kActCount)) &&
+               (gate_act == 0 || epilogue == kEpiSwiGLU || epilogue == kEpiActBF16),
                "gemm_tc: unknown epilogue %d (activation %d)", epilogue, gate_act);
     GI_REQUIRE(gate_up_bias == nullptr || epilogue == kEpiSwiGLU, "gemm_tc: a gate/up bias goes with the gated epilogue only");
-    const bool bf16_out = epilogue == kEpiSwiGLU;
+    const bool bf16_out = epilogue == kEpiSwiGLU || epilogue == kEpiActBF16;
     GI_REQUIRE((ldc * (bf16_out ? 2 : 4)) % 16 == 0, "gemm_tc: the output row stride %lld is not a multiple of 16 bytes", ldc);
     GI_REQUIRE((reinterpret_cast<uintptr_t>(A) % 16 == 0) && (reinterpret_cast<uintptr_t>(W) % 16 == 0) &&
                (reinterpret_cast<uintptr_t>(C) % 16 == 0), "gemm_tc: operands must be 16-byte aligned");
@@ -1768,7 +1800,7 @@ static int gi_gemm_tc_persistent_impl(const void* A, const void* W, void* C, int
     if (make_map(&mp, A, M, K, lda, kBlockP)) return 1;
     const bool split = splits > 1;
     if (split) {
-        GI_REQUIRE(epilogue != kEpiSwiGLU && N % 4 == 0 && splits <= 8, "gemm_tc: a split over K needs a 32-bit output, N %% 4 == 0 and at most 8 ranges");
+        GI_REQUIRE(!bf16_out && N % 4 == 0 && splits <= 8, "gemm_tc: a split over K needs a 32-bit output, N %% 4 == 0 and at most 8 ranges");
         p.kb_per_split = (total_kb + splits - 1) / splits;
         splits = (total_kb + p.kb_per_split - 1) / p.kb_per_split;             // every range holds at least one block
         p.splits = splits;
@@ -1797,6 +1829,11 @@ static int gi_gemm_tc_persistent_impl(const void* A, const void* W, void* C, int
     }
     p.tiles_q = (N + block_q - 1) / block_q;
     if (make_map(&mq, W, N, K, ldw, pair ? block_q / 2 : block_q)) return 1;
+    if (epilogue == kEpiActBF16) {
+        if (pair) return launch_persistent_pair<256, kEpiActBF16>(mp, mq, mc, p, st);
+        if (block_q == 256) return launch_persistent<256, kEpiActBF16>(mp, mq, mc, p, st);
+        return launch_persistent<128, kEpiActBF16>(mp, mq, mc, p, st);
+    }
     if (pair) {
         if (run_epilogue == kEpiAddF32) return launch_persistent_pair<256, kEpiAddF32>(mp, mq, mc, p, st);
         return finish(launch_persistent_pair<256, kEpiStoreF32>(mp, mq, mc, p, st));
@@ -1812,7 +1849,8 @@ static int gi_gemm_tc_persistent_impl(const void* A, const void* W, void* C, int
 // A matrix per group of rows: A [M, K] holds tiles of 128 rows each of which belongs to one group (an expert's tokens,
 // padded to whole tiles), W [groups * rows, K] the groups' matrices one after the other (rows = N, or 2 N = [gate; up]
 // with epilogue 2), tile_group[i] the group of tile i and *tiles_used how many tiles exist (device memory, written by
-// an earlier kernel). C [M, N] in the rows' order; epilogue 0 stores 32-bit, 2 stores act(gate) * up as bfloat16.
+// an earlier kernel). C [M, N] in the rows' order; epilogue 0 stores 32-bit, 2 stores act(gate) * up as bfloat16, 4
+// act(sum) as bfloat16.
 static int gi_gemm_tc_grouped_impl(const void* A, const void* W, void* C, int epilogue, int M, int N, int K, int groups,
                                   const int* tile_group, const int* tiles_used, void* status, float act_limit, void* stream) {
     if (M == 0 || N == 0) return 0;
@@ -1821,14 +1859,16 @@ static int gi_gemm_tc_grouped_impl(const void* A, const void* W, void* C, int ep
     GI_REQUIRE(K % 8 == 0, "gemm_tc grouped: K=%d must be a multiple of 8 (16-byte rows for TMA)", K);
     const int gate_act = epilogue >> 8;
     epilogue &= 0xff;
-    GI_REQUIRE((epilogue == kEpiStoreF32 || epilogue == kEpiSwiGLU) && gate_act >= 0 && gate_act < kActCount,
+    const bool gated = epilogue == kEpiSwiGLU;
+    GI_REQUIRE((epilogue == kEpiStoreF32 || gated || epilogue == kEpiActBF16) && gate_act >= 0 &&
+               gate_act < (gated ? static_cast<int>(kActCount) : static_cast<int>(kPlainCount)),
                "gemm_tc grouped: unknown epilogue %d (activation %d)", epilogue, gate_act);
-    const bool bf16_out = epilogue == kEpiSwiGLU;
+    const bool bf16_out = gated || epilogue == kEpiActBF16;
     GI_REQUIRE((static_cast<long long>(N) * (bf16_out ? 2 : 4)) % 16 == 0, "gemm_tc grouped: output rows of %d values are not a multiple of 16 bytes", N);
     GI_REQUIRE((reinterpret_cast<uintptr_t>(A) % 16 == 0) && (reinterpret_cast<uintptr_t>(W) % 16 == 0) &&
                (reinterpret_cast<uintptr_t>(C) % 16 == 0), "gemm_tc grouped: operands must be 16-byte aligned");
     GI_REQUIRE(status != nullptr && tile_group != nullptr && tiles_used != nullptr, "gemm_tc grouped: status word and tile lists are required");
-    const int block_q = (bf16_out ? N >= 128 : N >= 256) ? 256 : 128;
+    const int block_q = (gated ? N >= 128 : N >= 256) ? 256 : 128;
     TcPersistentParams p = {};
     p.rows_p = M; p.rows_q = N; p.K = K;
     p.tiles_p = M / kBlockP;
@@ -1836,14 +1876,14 @@ static int gi_gemm_tc_grouped_impl(const void* A, const void* W, void* C, int ep
     p.gate_act = gate_act; p.act_limit = act_limit; p.gate_up_bias = nullptr;
     p.status = static_cast<int*>(status);
     p.splits = 1; p.kb_per_split = (K + kBlockK - 1) / kBlockK; p.split_rows = 0;
-    p.tile_group = tile_group; p.tiles_used = tiles_used; p.group_rows = bf16_out ? 2 * N : N;
+    p.tile_group = tile_group; p.tiles_used = tiles_used; p.group_rows = gated ? 2 * N : N;
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     CUtensorMap mp, mq, mc;
     if (make_map(&mp, A, M, K, K, kBlockP)) return 1;
     if (make_out_map(&mc, C, M, N, N, bf16_out)) return 1;
     const long long w_rows = static_cast<long long>(groups) * p.group_rows;
     GI_REQUIRE(w_rows <= 2147483647LL, "gemm_tc grouped: too many weight rows");
-    if (bf16_out) {
+    if (gated) {
         p.tiles_q = (N + block_q / 2 - 1) / (block_q / 2);
         if (make_map(&mq, W, static_cast<int>(w_rows), K, K, block_q / 2)) return 1;
         if (block_q == 256) return launch_persistent<256, kEpiSwiGLU>(mp, mq, mc, p, st);
@@ -1851,6 +1891,10 @@ static int gi_gemm_tc_grouped_impl(const void* A, const void* W, void* C, int ep
     }
     p.tiles_q = (N + block_q - 1) / block_q;
     if (make_map(&mq, W, static_cast<int>(w_rows), K, K, block_q)) return 1;
+    if (bf16_out) {
+        if (block_q == 256) return launch_persistent<256, kEpiActBF16>(mp, mq, mc, p, st);
+        return launch_persistent<128, kEpiActBF16>(mp, mq, mc, p, st);
+    }
     if (block_q == 256) return launch_persistent<256, kEpiStoreF32>(mp, mq, mc, p, st);
     return launch_persistent<128, kEpiStoreF32>(mp, mq, mc, p, st);
 }

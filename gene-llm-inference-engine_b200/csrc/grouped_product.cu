@@ -9,8 +9,9 @@
 //              (32-bit, in a row of the token: the heads' outputs of a gated attention)
 //     experts  rows are (token, choice) pairs sorted by expert: tile i belongs to expert tile_group[i], its rows are
 //              sorted_rows[16 i ..] (-1: none); the input row is pair / a_div, the output row the pair;
-//              gated: out = act(W_gate a) * (W_up a) with W[g] = [gate rows; up rows]
-//   route             per token: z = W_r x in 32-bit, s = sigmoid(z), the ``top`` experts by s + correction, weights s
+//              gated: out = act(W_gate a) * (W_up a) with W[g] = [gate rows; up rows]; else optionally out = act(W a)
+//   route             per token: z = W_r x in 32-bit, s = sigmoid(z) or softmax(z) over all experts, the ``top`` experts by
+//                     s + correction; weights s, or s / (sum of the chosen s + 1e-20), times a constant
 //   route_align       buckets the pairs by expert into tiles of 16 rows (padding with -1), one block; for many rows
 //                     into tiles of 128, the token tiles of the tensor-core product that takes a matrix per tile
 //   gather_rows       a[r] = x[sorted_rows[r] / top] (zeros for padding): the rows in the tiles' order
@@ -35,6 +36,7 @@ struct GroupedArgs {
     int N, K, rows, groups;
     const int* tile_group; const int* sorted_rows; const int* n_tiles;   // experts form (else null)
     int act; float act_limit;                                     // gated: a GateAct code and its limit
+    int out_act;                                                  // not gated: a PlainAct code
     // rotated tail (heads form)
     int tail; const float* freq; float amplitude; const int* positions;
     // output gate (heads form): out *= sigmoid(gate[row, gate_off + h * N + n]), 32-bit (else null)
@@ -140,6 +142,7 @@ grouped_product_kernel(const GroupedArgs p) {
             if (n >= p.N) continue;
             float v = acc[i][j];
             if (GATED) v = gated_value(v, acc_up[U * i][j], p.act, p.act_limit);
+            else v = plain_value(v, p.out_act);
             v = gp_gated(p, v, r, g, n);
             const size_t o = static_cast<size_t>(r) * p.ldo + p.o_off + static_cast<size_t>(g) * p.o_gs + n;
             if (p.out_is_f32) static_cast<float*>(p.out)[o] = v;
@@ -267,6 +270,7 @@ grouped_rows_kernel(const GroupedArgs p) {
                 if (i < m_here && n_first + r < p.N) {
                     float v = warp_sum(acc[r][i]);
                     if (GATED) v = gated_value(v, warp_sum(acc_up[GATED ? r : 0][i]), p.act, p.act_limit);
+                    else v = plain_value(v, p.out_act);
                     if (p.gate != nullptr) v *= 1.0f / (1.0f + expf(-__shfl_sync(0xffffffffu, gate_z, r * kGrFew + i)));
                     if (lane == 0) {
                         const size_t o = static_cast<size_t>(s_row[m0 + i]) * p.ldo + p.o_off + static_cast<size_t>(g) * p.o_gs + n_first + r;
@@ -368,7 +372,7 @@ constexpr int kRouteMaxExperts = 1024;
 template <typename TX>
 __global__ void __launch_bounds__(128)
 route_kernel(const TX* __restrict__ x, int D, const float* __restrict__ w, const float* __restrict__ correction, int E, int top,
-             int* __restrict__ ids, float* __restrict__ weights) {
+             int softmax, int renormalise, float factor, int* __restrict__ ids, float* __restrict__ weights) {
     pdl_prologue();
     extern __shared__ float s_x[];                 // [D]
     __shared__ float s_score[kRouteMaxExperts], s_choice[kRouteMaxExperts];
@@ -381,13 +385,28 @@ route_kernel(const TX* __restrict__ x, int D, const float* __restrict__ w, const
         for (int d = lane; d < D; d += 32) z = fmaf(row[d], s_x[d], z);
         z = warp_sum(z);
         if (lane == 0) {
-            const float s = 1.0f / (1.0f + expf(-z));
+            const float s = softmax ? z : 1.0f / (1.0f + expf(-z));
             s_score[e] = s;
             s_choice[e] = s + (correction ? correction[e] : 0.f);
         }
     }
     __syncthreads();
     if (warp != 0) return;
+    if (softmax) {
+        float m = -INFINITY;
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, s_score[e]);
+        m = warp_max(m);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) sum += expf(s_score[e] - m);
+        const float inv = 1.0f / warp_sum(sum);
+        for (int e = lane; e < E; e += 32) {
+            const float s = expf(s_score[e] - m) * inv;
+            s_score[e] = s;
+            s_choice[e] = s + (correction ? correction[e] : 0.f);
+        }
+        __syncwarp();
+    }
+    float chosen = 0.f;
     // the ``top`` largest choice scores, the lowest index among equals; a chosen expert leaves the contest
     for (int k = 0; k < top; ++k) {
         float best = -INFINITY;
@@ -402,12 +421,18 @@ route_kernel(const TX* __restrict__ x, int D, const float* __restrict__ w, const
             const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
             if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
         }
+        if (best_e >= E) best_e = 0;                 // no comparable score (a row of NaN): any expert, but a real one
+        chosen += s_score[best_e];
         if (lane == 0) {
             ids[static_cast<size_t>(t) * top + k] = best_e;
-            weights[static_cast<size_t>(t) * top + k] = s_score[best_e];
+            weights[static_cast<size_t>(t) * top + k] = s_score[best_e] * factor;
             s_choice[best_e] = -INFINITY;
         }
         __syncwarp();
+    }
+    if (renormalise) {
+        const float inv = 1.0f / (chosen + 1e-20f);
+        for (int k = lane; k < top; k += 32) weights[static_cast<size_t>(t) * top + k] *= inv;
     }
 }
 
@@ -576,13 +601,14 @@ static int gi_expert_product_impl(const void* a, int a_dtype, long long lda, int
     if (max_tiles == 0) return 0;
     GI_REQUIRE(max_tiles > 0 && N > 0 && K > 0 && a_div > 0, "expert_product: sizes must be positive");
     GI_REQUIRE(tile_group && sorted_rows && n_tiles, "expert_product: the sorted rows are missing");
-    GI_REQUIRE(act >= 0 && act < kActCount, "expert_product: unknown activation code %d", act);
+    GI_REQUIRE(act >= 0 && act < (gated ? static_cast<int>(kActCount) : static_cast<int>(kPlainCount)), "expert_product: unknown activation code %d", act);
     GroupedArgs p = {};
     p.a = a; p.lda = lda; p.a_div = a_div;
     p.w = w; p.w_gs = w_gs; p.ldw = ldw; p.up_off = up_off;
     p.out = out; p.out_is_f32 = out_dtype == kF32; p.ldo = ldo;
     p.N = N; p.K = K; p.groups = 1;
-    p.tile_group = tile_group; p.sorted_rows = sorted_rows; p.n_tiles = n_tiles; p.act = act; p.act_limit = act_limit;
+    p.tile_group = tile_group; p.sorted_rows = sorted_rows; p.n_tiles = n_tiles; p.act = gated ? act : 0; p.act_limit = act_limit;
+    p.out_act = gated ? kPlainNone : act;
     dim3 grid(max_tiles, (N + kGpTN - 1) / kGpTN);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (rows_form_fits(p, a_dtype, w_dtype))
@@ -591,7 +617,7 @@ static int gi_expert_product_impl(const void* a, int a_dtype, long long lda, int
 }
 
 static int gi_route_impl(const void* x, int x_dtype, int T, int D, const float* w, const float* correction, int E, int top,
-                         int* ids, float* weights, int* sorted_rows, int* tile_group, int* n_tiles, int max_tiles, int tile_rows,
+                         int softmax, int renormalise, float factor, int* ids, float* weights, int* sorted_rows, int* tile_group, int* n_tiles, int max_tiles, int tile_rows,
                          int* pair_row, void* stream) {
     if (T == 0) return 0;
     GI_REQUIRE(T > 0 && D > 0 && E > 0 && top > 0 && top <= E, "route: sizes must be positive and top at most the experts");
@@ -604,10 +630,10 @@ static int gi_route_impl(const void* x, int x_dtype, int T, int D, const float* 
     const size_t smem = static_cast<size_t>(D) * 4;
     if (x_dtype == kF32) {
         if (smem > 40 * 1024) cudaFuncSetAttribute(route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-        launch_kernel((route_kernel<float>), dim3(T), dim3(128), smem, st, static_cast<const float*>(x), D, w, correction, E, top, ids, weights);
+        launch_kernel((route_kernel<float>), dim3(T), dim3(128), smem, st, static_cast<const float*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights);
     } else if (x_dtype == kBF16) {
         if (smem > 40 * 1024) cudaFuncSetAttribute(route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-        launch_kernel((route_kernel<__nv_bfloat16>), dim3(T), dim3(128), smem, st, static_cast<const __nv_bfloat16*>(x), D, w, correction, E, top, ids, weights);
+        launch_kernel((route_kernel<__nv_bfloat16>), dim3(T), dim3(128), smem, st, static_cast<const __nv_bfloat16*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights);
     } else {
         GI_REQUIRE(false, "route: unsupported dtype code %d", x_dtype);
     }
@@ -673,10 +699,10 @@ extern "C" int gi_expert_product(const void* a, int a_dtype, long long lda, int 
                         N, K, tile_group, sorted_rows, n_tiles, max_tiles, stream);
 }
 
-extern "C" int gi_route(const void* x, int x_dtype, int T, int D, const float* w, const float* correction, int E, int top, int* ids,
-                        float* weights, int* sorted_rows, int* tile_group, int* n_tiles, int max_tiles, int tile_rows, int* pair_row,
+extern "C" int gi_route(const void* x, int x_dtype, int T, int D, const float* w, const float* correction, int E, int top,
+                        int softmax, int renormalise, float factor, int* ids, float* weights, int* sorted_rows, int* tile_group, int* n_tiles, int max_tiles, int tile_rows, int* pair_row,
                         void* stream) {
-    return gi::dispatch(gi_route_impl, x, x_dtype, T, D, w, correction, E, top, ids, weights, sorted_rows, tile_group, n_tiles,
+    return gi::dispatch(gi_route_impl, x, x_dtype, T, D, w, correction, E, top, softmax, renormalise, factor, ids, weights, sorted_rows, tile_group, n_tiles,
                         max_tiles, tile_rows, pair_row, stream);
 }
 

@@ -1,5 +1,6 @@
 // Kernels of layers whose mixer and feed-forward read one normed input and are added together, of a residual stream
-// that is a weighted mix of all earlier layers' results, and a few small element-wise steps around them.
+// that is a weighted mix of all earlier layers' results or is replaced by a product over itself and the embedding, and a
+// few small element-wise steps around them.
 //
 //   add_rows_at     x[t, :] += table[index[t], :]: a learned vector per position added to the embedding
 //   add_bias        y[t, :] += b: the bias of a product that adds into a stream
@@ -8,8 +9,13 @@
 //                   x the stream that layer i read and y what its sublayers produced:
 //                   h[t, i + 1] = x[t] + m (y[t] + b);  x[t] = sum_{j <= i + 1} w[j] h[t, j]   (w: the layer's i + 2 mixing
 //                   weights; b: an optional bias that a sublayer's last product left to this kernel);
-//                   without weights x[t] += m (y[t] + b). The same pass clears y and writes the unit-RMS norm of the new x
-//                   times one number (the next layer's single norm weight) in the compute dtype.
+//                   without weights x[t] += m (y[t] + b). The same pass clears y and writes what runs next reads, in the
+//                   compute dtype: the unit-RMS norm of the new x times one number (the next layer's single norm weight); its
+//                   layer norm (next_weight and next_bias of D values each); or, when a product over the stream itself comes
+//                   next (``handover``), the new x as it is, the stream then starting again from handover[t]
+//   layer_norm      out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b per row
+//   take_stream     xn = x in the compute dtype and x = from: what a product that replaces the stream reads and adds to
+//   plain_act       out = act(z): the activation of an ungated feed-forward where no product's epilogue applies it
 //   softcap         z <- cap * tanh(z / cap), in place
 //
 // All arithmetic is 32-bit; only stores to a bfloat16 output round. A row's result depends on that row only.
@@ -96,11 +102,97 @@ template <int VEC, typename TOut> __device__ __forceinline__ void store_piece_as
 // i of thread t at (i * 256 + t) * VEC. The sum over the slots runs in slot order; the row's sum of squares is each
 // thread's chain over its pieces, added by a fixed xor tree and then over the warps in index order: a row's result
 // depends on that row only. The first kDepthKept pieces of a thread stay in registers for the second pass.
+__device__ __forceinline__ float block_sum_of_256(float v, float* warp_part) {
+    v = warp_sum(v);
+    __syncthreads();                                    // the sum before has been read
+    if ((threadIdx.x & 31) == 0) warp_part[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float total = 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) total += warp_part[k];
+    return total;
+}
+
+// One block per row, pieces of VEC values, the first kDepthKept of a thread in registers through the three passes (mean,
+// variance, result). Sums: a thread's chain, a fixed xor tree, the warps in index order.
+template <typename TOut, int VEC>
+__global__ void __launch_bounds__(256)
+layer_norm_kernel(const float* __restrict__ x, const int* __restrict__ rows, const float* __restrict__ weight,
+                  const float* __restrict__ bias, TOut* __restrict__ out, int D, float eps) {
+    pdl_prologue();
+    __shared__ float warp_part[8];
+    const float* xr = x + static_cast<size_t>(rows ? rows[blockIdx.x] : static_cast<int>(blockIdx.x)) * D;
+    TOut* o = out + static_cast<size_t>(blockIdx.x) * D;
+    Piece<VEC> keep[kDepthKept];
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kDepthKept; ++i) {
+        const int d = (i * 256 + threadIdx.x) * VEC;
+        if (d < D) {
+            keep[i] = load_piece<VEC>(xr + d);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) sum += keep[i].v[e];
+        }
+    }
+    for (int d = (kDepthKept * 256 + threadIdx.x) * VEC; d < D; d += 256 * VEC) {
+        const Piece<VEC> v = load_piece<VEC>(xr + d);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) sum += v.v[e];
+    }
+    const float mean = block_sum_of_256(sum, warp_part) / static_cast<float>(D);
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kDepthKept; ++i) {
+        if ((i * 256 + threadIdx.x) * VEC < D) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss = fmaf(keep[i].v[e] - mean, keep[i].v[e] - mean, ss);
+        }
+    }
+    for (int d = (kDepthKept * 256 + threadIdx.x) * VEC; d < D; d += 256 * VEC) {
+        const Piece<VEC> v = load_piece<VEC>(xr + d);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ss = fmaf(v.v[e] - mean, v.v[e] - mean, ss);
+    }
+    const float scale = 1.0f / sqrtf(block_sum_of_256(ss, warp_part) / static_cast<float>(D) + eps);
+    auto finish = [&](int d, const Piece<VEC>& v) {
+        const Piece<VEC> w = load_piece<VEC>(weight + d), b = load_piece<VEC>(bias + d);
+        Piece<VEC> r;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) r.v[e] = fmaf(scale * (v.v[e] - mean), w.v[e], b.v[e]);
+        store_piece_as<VEC, TOut>(o + d, r);
+    };
+#pragma unroll
+    for (int i = 0; i < kDepthKept; ++i) {
+        const int d = (i * 256 + threadIdx.x) * VEC;
+        if (d < D) finish(d, keep[i]);
+    }
+    for (int d = (kDepthKept * 256 + threadIdx.x) * VEC; d < D; d += 256 * VEC) finish(d, load_piece<VEC>(xr + d));
+}
+
+template <typename TOut>
+__global__ void __launch_bounds__(256)
+plain_act_kernel(const float* __restrict__ z, TOut* __restrict__ out, int act, size_t total) {
+    pdl_prologue();
+    for (size_t i = static_cast<size_t>(blockIdx.x) * 256 + threadIdx.x; i < total; i += static_cast<size_t>(gridDim.x) * 256)
+        out[i] = from_float<TOut>(plain_value(z[i], act));
+}
+
+template <typename TOut>
+__global__ void __launch_bounds__(256)
+take_stream_kernel(float* __restrict__ x, const float* __restrict__ from, TOut* __restrict__ xn, size_t total) {
+    pdl_prologue();
+    for (size_t i = static_cast<size_t>(blockIdx.x) * 256 + threadIdx.x; i < total; i += static_cast<size_t>(gridDim.x) * 256) {
+        const float v = x[i];
+        x[i] = from[i];
+        xn[i] = from_float<TOut>(v);
+    }
+}
+
 template <typename TOut, int VEC>
 __global__ void __launch_bounds__(256)
 depth_mix_kernel(float* __restrict__ x, float* __restrict__ y, const float* __restrict__ y_bias, float m, float* __restrict__ hist, int slots, int slot,
-                 const float* __restrict__ w, int first, const float* __restrict__ next_weight, float eps,
-                 TOut* __restrict__ xn_out, int D) {
+                 const float* __restrict__ w, int first, const float* __restrict__ next_weight, const float* __restrict__ next_bias,
+                 const float* __restrict__ handover, float eps, TOut* __restrict__ xn_out, int D) {
     pdl_prologue();
     __shared__ float warp_part[8];
     __shared__ float s_w[kDepthWeights];
@@ -111,7 +203,7 @@ depth_mix_kernel(float* __restrict__ x, float* __restrict__ y, const float* __re
         __syncthreads();
     }
     Piece<VEC> keep[kDepthKept];
-    float ss = 0.f;
+    float ss = 0.f, sum = 0.f;
 
     // what a piece reads: the stream, the sublayers' sum (with the bias) and the weighted sum of the kept results before
     // this layer's, in slot order (slot 0 is the stream itself while the history is still empty)
@@ -148,9 +240,14 @@ depth_mix_kernel(float* __restrict__ x, float* __restrict__ y, const float* __re
 #pragma unroll
             for (int e = 0; e < VEC; ++e) v.v[e] = fmaf(ws, fresh.v[e], acc.v[e]);
         }
+        if (handover) {
+            store_piece<VEC>(x + row + d, load_piece<VEC>(handover + row + d));
+            store_piece_as<VEC, TOut>(xn_out + row + d, v);
+            return v;
+        }
         store_piece<VEC>(x + row + d, v);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) ss = fmaf(v.v[e], v.v[e], ss);
+        for (int e = 0; e < VEC; ++e) { ss = fmaf(v.v[e], v.v[e], ss); sum += v.v[e]; }
         return v;
     };
 
@@ -172,7 +269,38 @@ depth_mix_kernel(float* __restrict__ x, float* __restrict__ y, const float* __re
         read(d, xo, yy, acc);
         write(d, xo, yy, acc);
     }
-    if (xn_out == nullptr) return;
+    if (xn_out == nullptr || handover) return;
+    if (next_bias) {                                    // a layer norm: mean, then the mean of the squared deviations
+        const float mean = block_sum_of_256(sum, warp_part) / static_cast<float>(D);
+        ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < kDepthKept; ++i) {
+            if ((i * 256 + threadIdx.x) * VEC < D) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) ss = fmaf(keep[i].v[e] - mean, keep[i].v[e] - mean, ss);
+            }
+        }
+        for (int d = (kDepthKept * 256 + threadIdx.x) * VEC; d < D; d += 256 * VEC) {
+            const Piece<VEC> v = load_piece<VEC>(x + row + d);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) ss = fmaf(v.v[e] - mean, v.v[e] - mean, ss);
+        }
+        const float scale = 1.0f / sqrtf(block_sum_of_256(ss, warp_part) / static_cast<float>(D) + eps);
+        auto finish = [&](int d, const Piece<VEC>& v) {
+            const Piece<VEC> nw = load_piece<VEC>(next_weight + d), nb = load_piece<VEC>(next_bias + d);
+            Piece<VEC> o;
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) o.v[e] = fmaf(scale * (v.v[e] - mean), nw.v[e], nb.v[e]);
+            store_piece_as<VEC, TOut>(xn_out + row + d, o);
+        };
+#pragma unroll
+        for (int i = 0; i < kDepthKept; ++i) {
+            const int d = (i * 256 + threadIdx.x) * VEC;
+            if (d < D) finish(d, keep[i]);
+        }
+        for (int d = (kDepthKept * 256 + threadIdx.x) * VEC; d < D; d += 256 * VEC) finish(d, load_piece<VEC>(x + row + d));
+        return;
+    }
     ss = warp_sum(ss);
     if ((threadIdx.x & 31) == 0) warp_part[threadIdx.x >> 5] = ss;
     __syncthreads();
@@ -258,25 +386,29 @@ static int gi_scale_impl(float* z, long long total, float factor, void* stream) 
 }
 
 static int gi_depth_mix_impl(float* x, float* y, const float* y_bias, float m, float* hist, int slots, int slot, const float* w, int first,
-                             const float* next_weight, float eps, void* xn_out, int xn_dtype, int T, int D, void* stream) {
+                             const float* next_weight, const float* next_bias, const float* handover, float eps, void* xn_out, int xn_dtype,
+                             int T, int D, void* stream) {
     if (T == 0) return 0;
     GI_REQUIRE(T > 0 && D > 0, "depth_mix: sizes must be positive");
+    GI_REQUIRE((next_bias == nullptr || next_weight != nullptr) && (handover == nullptr || (xn_out != nullptr && next_bias == nullptr)),
+               "depth_mix: a layer norm needs its weight, a hand-over a place for the stream and no norm");
     GI_REQUIRE(hist == nullptr || (w != nullptr && slot >= 1 && slot < slots), "depth_mix: slot %d lies outside the %d kept results", slot, slots);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
-    const bool vec = D % 4 == 0 && aligned(x) && aligned(y) && aligned(hist) && aligned(y_bias) && aligned(xn_out);
+    const bool vec = D % 4 == 0 && aligned(x) && aligned(y) && aligned(hist) && aligned(y_bias) && aligned(xn_out) &&
+                     aligned(handover) && aligned(next_bias) && (next_bias == nullptr || aligned(next_weight));
     GI_REQUIRE(xn_dtype == kBF16 || xn_dtype == kF32, "depth_mix: unsupported dtype code %d", xn_dtype);
     if (xn_dtype == kBF16 && vec)
-        launch_kernel((depth_mix_kernel<__nv_bfloat16, 4>), dim3(T), dim3(256), 0, st, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, eps,
+        launch_kernel((depth_mix_kernel<__nv_bfloat16, 4>), dim3(T), dim3(256), 0, st, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, next_bias, handover, eps,
                       static_cast<__nv_bfloat16*>(xn_out), D);
     else if (xn_dtype == kBF16)
-        launch_kernel((depth_mix_kernel<__nv_bfloat16, 1>), dim3(T), dim3(256), 0, st, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, eps,
+        launch_kernel((depth_mix_kernel<__nv_bfloat16, 1>), dim3(T), dim3(256), 0, st, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, next_bias, handover, eps,
                       static_cast<__nv_bfloat16*>(xn_out), D);
     else if (vec)
-        launch_kernel((depth_mix_kernel<float, 4>), dim3(T), dim3(256), 0, st, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, eps,
+        launch_kernel((depth_mix_kernel<float, 4>), dim3(T), dim3(256), 0, st, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, next_bias, handover, eps,
                       static_cast<float*>(xn_out), D);
     else
-        launch_kernel((depth_mix_kernel<float, 1>), dim3(T), dim3(256), 0, st, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, eps,
+        launch_kernel((depth_mix_kernel<float, 1>), dim3(T), dim3(256), 0, st, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, next_bias, handover, eps,
                       static_cast<float*>(xn_out), D);
     return check_launch("depth_mix");
 }
@@ -302,6 +434,60 @@ extern "C" int gi_scale(float* z, long long total, float factor, void* stream) {
 }
 
 extern "C" int gi_depth_mix(float* x, float* y, const float* y_bias, float m, float* hist, int slots, int slot, const float* w, int first,
-                            const float* next_weight, float eps, void* xn_out, int xn_dtype, int T, int D, void* stream) {
-    return gi::dispatch(gi_depth_mix_impl, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, eps, xn_out, xn_dtype, T, D, stream);
+                            const float* next_weight, const float* next_bias, const float* handover, float eps, void* xn_out, int xn_dtype,
+                            int T, int D, void* stream) {
+    return gi::dispatch(gi_depth_mix_impl, x, y, y_bias, m, hist, slots, slot, w, first, next_weight, next_bias, handover, eps, xn_out, xn_dtype, T, D, stream);
+}
+
+static int gi_layer_norm_impl(const float* x, const int* rows, const float* weight, const float* bias, void* out, int out_dtype, int n, int D,
+                              float eps, void* stream) {
+    if (n == 0) return 0;
+    GI_REQUIRE(n > 0 && D > 0, "layer_norm: sizes must be positive (rows=%d, D=%d)", n, D);
+    GI_REQUIRE(out_dtype == kBF16 || out_dtype == kF32, "layer_norm: unsupported dtype code %d", out_dtype);
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+    const bool vec = D % 4 == 0 && aligned(x) && aligned(weight) && aligned(bias) && aligned(out);
+    if (out_dtype == kBF16 && vec)
+        launch_kernel((layer_norm_kernel<__nv_bfloat16, 4>), dim3(n), dim3(256), 0, st, x, rows, weight, bias, static_cast<__nv_bfloat16*>(out), D, eps);
+    else if (out_dtype == kBF16)
+        launch_kernel((layer_norm_kernel<__nv_bfloat16, 1>), dim3(n), dim3(256), 0, st, x, rows, weight, bias, static_cast<__nv_bfloat16*>(out), D, eps);
+    else if (vec)
+        launch_kernel((layer_norm_kernel<float, 4>), dim3(n), dim3(256), 0, st, x, rows, weight, bias, static_cast<float*>(out), D, eps);
+    else
+        launch_kernel((layer_norm_kernel<float, 1>), dim3(n), dim3(256), 0, st, x, rows, weight, bias, static_cast<float*>(out), D, eps);
+    return check_launch("layer_norm");
+}
+
+static int gi_take_stream_impl(float* x, const float* from, void* xn, int xn_dtype, long long total, void* stream) {
+    if (total == 0) return 0;
+    GI_REQUIRE(total > 0, "take_stream: the size must be positive");
+    GI_REQUIRE(xn_dtype == kBF16 || xn_dtype == kF32, "take_stream: unsupported dtype code %d", xn_dtype);
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const dim3 grid(grid_for(static_cast<size_t>(total)));
+    if (xn_dtype == kBF16) launch_kernel((take_stream_kernel<__nv_bfloat16>), grid, dim3(256), 0, st, x, from, static_cast<__nv_bfloat16*>(xn), static_cast<size_t>(total));
+    else launch_kernel((take_stream_kernel<float>), grid, dim3(256), 0, st, x, from, static_cast<float*>(xn), static_cast<size_t>(total));
+    return check_launch("take_stream");
+}
+
+static int gi_plain_act_impl(const float* z, void* out, int out_dtype, long long total, int act, void* stream) {
+    if (total == 0) return 0;
+    GI_REQUIRE(total > 0 && act >= 0 && act < kPlainCount, "plain_act: unknown activation code %d", act);
+    GI_REQUIRE(out_dtype == kBF16 || out_dtype == kF32, "plain_act: unsupported dtype code %d", out_dtype);
+    cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const dim3 grid(grid_for(static_cast<size_t>(total)));
+    if (out_dtype == kBF16) launch_kernel((plain_act_kernel<__nv_bfloat16>), grid, dim3(256), 0, st, z, static_cast<__nv_bfloat16*>(out), act, static_cast<size_t>(total));
+    else launch_kernel((plain_act_kernel<float>), grid, dim3(256), 0, st, z, static_cast<float*>(out), act, static_cast<size_t>(total));
+    return check_launch("plain_act");
+}
+
+extern "C" int gi_plain_act(const float* z, void* out, int out_dtype, long long total, int act, void* stream) {
+    return gi::dispatch(gi_plain_act_impl, z, out, out_dtype, total, act, stream);
+}
+
+extern "C" int gi_layer_norm(const float* x, const int* rows, const float* weight, const float* bias, void* out, int out_dtype, int n, int D, float eps, void* stream) {
+    return gi::dispatch(gi_layer_norm_impl, x, rows, weight, bias, out, out_dtype, n, D, eps, stream);
+}
+
+extern "C" int gi_take_stream(float* x, const float* from, void* xn, int xn_dtype, long long total, void* stream) {
+    return gi::dispatch(gi_take_stream_impl, x, from, xn, xn_dtype, total, stream);
 }

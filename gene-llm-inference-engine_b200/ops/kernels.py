@@ -193,6 +193,10 @@ def rope_store(qkv: torch.Tensor, positions: torch.Tensor, row_req: torch.Tensor
 ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "capped_swish": 3}
 
 
+# what an ungated feed-forward applies to its first product: nothing, or relu(z)^2
+PLAIN_ACTIVATIONS = {"none": 0, "relu2": 1}
+
+
 def scale_cast(x: torch.Tensor, acc: torch.Tensor, xn: Optional[torch.Tensor], alpha: float) -> None:
     """acc = alpha * x (32-bit) and, when given, xn = x in xn's dtype."""
     if acc.shape != x.shape or (xn is not None and xn.shape != x.shape):
@@ -264,6 +268,48 @@ def norm_rope_store(proj: torch.Tensor, q_offset: int, k_offset: int, v_offset: 
         head_dim, vd, page_size, int(write_kv), int(bool(wide_norm)), _stream()), "norm_rope_store")
 
 
+def maps_norm_store(proj: torch.Tensor, q_offset: int, k_offset: int, v_offset: int, q_norm: torch.Tensor, k_norm: torch.Tensor,
+                    eps: float, temperature, positions: torch.Tensor, row_req: torch.Tensor, block_tables: torch.Tensor,
+                    q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, num_heads: int, num_kv_heads: int, dim: int,
+                    value_dim: int, page_size: int, write_kv: bool = True) -> None:
+    """Heads of two score maps: from the 32-bit projections ``proj`` [T, ld] (from q_offset H heads of [map 1, map 2], dim
+    values each; from k_offset G such heads; from v_offset G value heads), every map is brought to unit RMS and weighted by
+    ``q_norm`` / ``k_norm`` [dim]; with ``temperature`` (coef, every) the queries at position p are multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1). ``q_out`` [T, H * 2 * 2 dim]: row [map 1, 0], then row [0, map 2] per head; keys
+    into the token's row of ``k_cache`` [pages, G, page_size, 2 dim], values into ``v_cache`` [pages, G, page_size, value_dim]."""
+    T, ld = proj.shape
+    if q_out.shape != (T, num_heads * 4 * dim):
+        raise KernelError("maps_norm_store: q_out must be [T, H * 2 * 2 dim]")
+    if k_cache.dtype != q_out.dtype or v_cache.dtype != q_out.dtype:
+        raise KernelError("maps_norm_store: q_out and the cache must have one dtype")
+    if k_cache.shape[1:] != (num_kv_heads, page_size, 2 * dim) or v_cache.shape != (k_cache.shape[0], num_kv_heads, page_size, value_dim):
+        raise KernelError("maps_norm_store: the cache must be [pages, G, page_size, 2 dim] (values: their own width)")
+    if q_norm.numel() != dim or k_norm.numel() != dim:
+        raise KernelError("maps_norm_store: the norms' weights must have dim values")
+    coef, every = temperature if temperature is not None else (0.0, 1.0)
+    check(lib().gi_maps_norm_store(
+        _dev(proj, "proj", torch.float32), ld, int(q_offset), int(k_offset), int(v_offset), _dev(q_norm, "q_norm", torch.float32),
+        _dev(k_norm, "k_norm", torch.float32), float(eps), float(coef), float(every), _dev(positions, "positions", torch.int32),
+        _dev(row_req, "row_req", torch.int32), _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1],
+        _dev(q_out, "q_out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), dtype_code(q_out.dtype), T, num_heads, num_kv_heads,
+        dim, value_dim, page_size, int(write_kv), _stream()), "maps_norm_store")
+
+
+def maps_combine_supported(value_dim: int) -> bool:
+    return value_dim <= 512
+
+
+def maps_combine(a: torch.Tensor, out: torch.Tensor, weight: float, eps: float, factor: float, num_heads: int) -> None:
+    """``a`` [T, H * 2 * vd] holds two outputs a1, a2 per head: out[t, h] = factor * N(a1 - weight * a2), N to unit RMS over the
+    vd values."""
+    T = a.shape[0]
+    vd = out.shape[1] // num_heads
+    if out.shape != (T, num_heads * vd) or a.shape != (T, 2 * num_heads * vd):
+        raise KernelError("maps_combine: a must be [T, H * 2 * vd] for out [T, H * vd]")
+    check(lib().gi_maps_combine(_dev(a, "a"), dtype_code(a.dtype), _dev(out, "out"), dtype_code(out.dtype), float(weight), float(eps),
+                                float(factor), T, num_heads, vd, _stream()), "maps_combine")
+
+
 def add_normed(y: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, eps: float, xn_out: Optional[torch.Tensor] = None,
                clear_y: bool = False) -> None:
     """x += weight * (y / sqrt(mean(y^2) + eps)) per row, in 32-bit; optionally also xn_out = x in xn_out's dtype and
@@ -283,6 +329,14 @@ def add_rows_at(x: torch.Tensor, table: torch.Tensor, index: torch.Tensor) -> No
         raise KernelError("add_rows_at: shapes of x, table and index do not agree")
     check(lib().gi_add_rows_at(_dev(x, "x", torch.float32), _dev(table, "table"), dtype_code(table.dtype), _dev(index, "index", torch.int32),
                                T, D, table.shape[0], _stream()), "add_rows_at")
+
+
+def plain_act(z: torch.Tensor, out: torch.Tensor, act: str) -> None:
+    """out = act(z) for act in PLAIN_ACTIVATIONS; z 32-bit, out 32-bit or bfloat16."""
+    if out.shape != z.shape or act not in PLAIN_ACTIVATIONS:
+        raise KernelError(f"plain_act: shapes do not agree or the activation '{act}' is unknown")
+    check(lib().gi_plain_act(_dev(z, "z", torch.float32), _dev(out, "out"), dtype_code(out.dtype), z.numel(), PLAIN_ACTIVATIONS[act],
+                             _stream()), "plain_act")
 
 
 def add_bias(y: torch.Tensor, bias: torch.Tensor) -> None:
@@ -314,14 +368,21 @@ def scale(z: torch.Tensor, factor: float) -> None:
 
 def depth_mix(x: torch.Tensor, y: torch.Tensor, mult: float, history: Optional[torch.Tensor] = None, slot: int = 0,
               weights: Optional[torch.Tensor] = None, first: bool = False, next_weight: Optional[torch.Tensor] = None,
-              eps: float = 0.0, xn_out: Optional[torch.Tensor] = None, y_bias: Optional[torch.Tensor] = None) -> None:
+              eps: float = 0.0, xn_out: Optional[torch.Tensor] = None, y_bias: Optional[torch.Tensor] = None,
+              next_bias: Optional[torch.Tensor] = None, handover: Optional[torch.Tensor] = None) -> None:
     """The end of a layer whose sublayers were summed into ``y``: fresh = x + mult * y and y = 0 (``y_bias`` [D]: a bias
     that a sublayer's last product left to this kernel, added to every row of y first). With ``history``
     [T, slots, D] (every layer's fresh result, slot 0 what the first layer read: written too when ``first``) and
     ``weights`` [slot + 1]: history[:, slot] = fresh and x = sum_j weights[j] * history[:, j] over j <= slot; without,
     x = fresh. ``xn_out``: also next_weight[0] * x / sqrt(mean(x^2) + eps) in xn_out's dtype (the next layer's normed
-    input when its norm has a single weight)."""
+    input when its norm has a single weight); with ``next_bias`` [D] (then ``next_weight`` [D] too) the layer norm of x
+    instead; with ``handover`` [T, D] xn_out = x itself and x = handover (a product over the stream comes next, whose
+    output is added to ``handover``)."""
     T, D = x.shape
+    if next_bias is not None and (next_bias.numel() != D or next_weight is None or next_weight.numel() != D or xn_out is None):
+        raise KernelError("depth_mix: a layer norm needs a weight and a bias per column and a place for its output")
+    if handover is not None and (handover.shape != x.shape or xn_out is None or next_bias is not None):
+        raise KernelError("depth_mix: a hand-over needs a place for the stream and comes without a norm")
     if y.shape != x.shape or (xn_out is not None and xn_out.shape != x.shape) or (y_bias is not None and y_bias.numel() != D):
         raise KernelError("depth_mix: shapes do not agree")
     slots = 0
@@ -331,8 +392,30 @@ def depth_mix(x: torch.Tensor, y: torch.Tensor, mult: float, history: Optional[t
         slots = history.shape[1]
     check(lib().gi_depth_mix(_dev(x, "x", torch.float32), _dev(y, "y", torch.float32), _opt(y_bias, "y_bias", torch.float32), float(mult), _opt(history, "history", torch.float32),
                              slots, int(slot), _opt(weights, "weights", torch.float32), int(bool(first)),
-                             _opt(next_weight, "next_weight", torch.float32), float(eps), 0 if xn_out is None else _dev(xn_out, "xn_out"),
+                             _opt(next_weight, "next_weight", torch.float32), _opt(next_bias, "next_bias", torch.float32),
+                             _opt(handover, "handover", torch.float32), float(eps), 0 if xn_out is None else _dev(xn_out, "xn_out"),
                              F32 if xn_out is None else dtype_code(xn_out.dtype), T, D, _stream()), "depth_mix")
+
+
+def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out: torch.Tensor, eps: float,
+               rows: Optional[torch.Tensor] = None) -> None:
+    """out[r, :] = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias of row r of x (of row rows[r] with ``rows``)."""
+    n, D = out.shape
+    if x.shape[1] != D or weight.numel() != D or bias.numel() != D:
+        raise KernelError("layer_norm: shapes of x, weight, bias and out do not agree")
+    if (rows is None and x.shape[0] < n) or (rows is not None and rows.numel() != n):
+        raise KernelError("layer_norm: rows and out do not agree")
+    check(lib().gi_layer_norm(_dev(x, "x", torch.float32), _opt(rows, "rows", torch.int32), _dev(weight, "weight", torch.float32),
+                              _dev(bias, "bias", torch.float32), _dev(out, "out"), dtype_code(out.dtype), n, D, float(eps), _stream()),
+          "layer_norm")
+
+
+def take_stream(x: torch.Tensor, start: torch.Tensor, xn: torch.Tensor) -> None:
+    """xn = x in xn's dtype and x = start, 32-bit: what a product that replaces the stream reads and adds to."""
+    if start.shape != x.shape or xn.shape != x.shape:
+        raise KernelError("take_stream: shapes do not agree")
+    check(lib().gi_take_stream(_dev(x, "x", torch.float32), _dev(start, "start", torch.float32), _dev(xn, "xn"), dtype_code(xn.dtype),
+                               x.numel(), _stream()), "take_stream")
 
 
 def streams(X: torch.Tensor, single: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None, clear_y: bool = False,
@@ -557,9 +640,11 @@ def route_tiles(n_tokens: int, top: int, experts: int, tile_rows: Optional[int] 
 
 def route(x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tensor], top: int, ids: torch.Tensor,
           weights: torch.Tensor, sorted_rows: torch.Tensor, tile_group: torch.Tensor, n_tiles: torch.Tensor,
-          tile_rows: Optional[int] = None, pair_row: Optional[torch.Tensor] = None) -> None:
-    """Per row of ``x`` [T, D]: s = sigmoid(w x) with ``w`` [E, D] 32-bit; the ``top`` experts with the largest
-    s + correction go to ``ids`` [T, top] and their s to ``weights`` [T, top]. The pairs (token, choice) are then
+          tile_rows: Optional[int] = None, pair_row: Optional[torch.Tensor] = None, scores: str = "sigmoid",
+          renormalise: bool = False, factor: float = 1.0) -> None:
+    """Per row of ``x`` [T, D]: s = sigmoid(w x) with ``w`` [E, D] 32-bit (``scores`` "softmax": s = softmax(w x) over all
+    experts); the ``top`` experts with the largest s + correction go to ``ids`` [T, top] and their s to ``weights`` [T, top]
+    (``renormalise``: divided by the chosen ones' sum + 1e-20), times ``factor``. The pairs (token, choice) are then
     bucketed by expert into tiles of ``tile_rows`` rows (grouped_tile_rows() by default): ``sorted_rows`` (pair index
     or -1), ``tile_group`` (a tile's expert), ``n_tiles`` [1], and optionally ``pair_row`` [T * top], the row each pair
     landed in. Two launches."""
@@ -571,8 +656,10 @@ def route(x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tensor], 
         raise KernelError("route: shapes do not agree")
     if sorted_rows.numel() < max_tiles * tm or max_tiles < route_tiles(T, top, E, tm) or (pair_row is not None and pair_row.numel() < T * top):
         raise KernelError("route: the buffers of the tiles are too small")
+    if scores not in ("sigmoid", "softmax"):
+        raise KernelError(f"route: unknown scores '{scores}'")
     check(lib().gi_route(_dev(x, "x"), dtype_code(x.dtype), T, D, _dev(w, "w", torch.float32), _opt(correction, "correction", torch.float32),
-                         E, int(top), _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32),
+                         E, int(top), int(scores == "softmax"), int(bool(renormalise)), float(factor), _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32),
                          _dev(sorted_rows, "sorted_rows", torch.int32), _dev(tile_group, "tile_group", torch.int32),
                          _dev(n_tiles, "n_tiles", torch.int32), max_tiles, tm, _opt(pair_row, "pair_row", torch.int32), _stream()), "route")
     count_launches(1)
@@ -608,10 +695,13 @@ def gather_rows(x: torch.Tensor, a_div: int, sorted_rows: torch.Tensor, n_tiles:
 
 
 def expert_product_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_group: torch.Tensor, n_tiles: torch.Tensor,
-                      gated: Optional[str] = None, limit: float = 0.0) -> None:
+                      gated: Optional[str] = None, limit: float = 0.0, act: Optional[str] = None) -> None:
     """The same on the tensor cores (bfloat16) for rows already in the tiles' order: ``a`` [tiles * 128, K], tile i
-    multiplies ``w[tile_group[i]]``; ``out`` [tiles * 128, N] 32-bit, or gated: bfloat16 act(gate) * up."""
+    multiplies ``w[tile_group[i]]``; ``out`` [tiles * 128, N] 32-bit, or bfloat16: gated act(gate) * up, or with ``act`` (one
+    of PLAIN_ACTIVATIONS) act of the product."""
     E, rows, K = w.shape
+    if act is not None and (gated is not None or act not in PLAIN_ACTIVATIONS):
+        raise KernelError(f"expert_product_tc: unknown activation '{act}' (or one beside a gated one)")
     N = rows // 2 if gated else rows
     M = a.shape[0]
     if a.shape != (M, K) or out.shape != (M, N) or M % TC_TILE_ROWS or tile_group.numel() < M // TC_TILE_ROWS:
@@ -620,8 +710,8 @@ def expert_product_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_
         raise KernelError(f"expert_product_tc: unknown activation '{gated}'")
     st = _tc_state(a.device)
     check(lib().gi_gemm_tc_grouped(_dev(a, "a", torch.bfloat16), _dev(w, "w", torch.bfloat16),
-                                   _dev(out, "out", torch.bfloat16 if gated else torch.float32),
-                                   (2 | (ACTIVATIONS[gated] << 8)) if gated else 0, M, N, K, E,
+                                   _dev(out, "out", torch.bfloat16 if gated or act else torch.float32),
+                                   (2 | (ACTIVATIONS[gated] << 8)) if gated else (4 | (PLAIN_ACTIVATIONS[act] << 8)) if act else 0, M, N, K, E,
                                    _dev(tile_group, "tile_group", torch.int32), _dev(n_tiles, "n_tiles", torch.int32),
                                    st.status.data_ptr(), float(limit), _stream()), "expert_product_tc")
 
@@ -632,9 +722,13 @@ def expert_product_tc_supported(N: int, K: int, gated: bool) -> bool:
 
 
 def expert_product(a: torch.Tensor, a_div: int, w: torch.Tensor, out: torch.Tensor, sorted_rows: torch.Tensor,
-                   tile_group: torch.Tensor, n_tiles: torch.Tensor, gated: Optional[str] = None, limit: float = 0.0) -> None:
+                   tile_group: torch.Tensor, n_tiles: torch.Tensor, gated: Optional[str] = None, limit: float = 0.0,
+                   act: Optional[str] = None) -> None:
     """out[pair] = W[expert of pair] a[pair // a_div] for the pairs that ``route`` bucketed, ``w`` [E, N, K] (gated:
-    [E, 2N, K], gate rows first, and out = act(gate) * up with ``gated`` one of ACTIVATIONS)."""
+    [E, 2N, K], gate rows first, and out = act(gate) * up with ``gated`` one of ACTIVATIONS). ``act``: one of
+    PLAIN_ACTIVATIONS on the output of an ungated product."""
+    if act is not None and (gated is not None or act not in PLAIN_ACTIVATIONS):
+        raise KernelError(f"expert_product: unknown activation '{act}' (or one beside a gated one)")
     E, rows, K = w.shape
     N = rows // 2 if gated else rows
     if a.dim() != 2 or a.shape[1] != K or out.dim() != 2 or out.shape[1] != N:
@@ -642,7 +736,8 @@ def expert_product(a: torch.Tensor, a_div: int, w: torch.Tensor, out: torch.Tens
     if gated is not None and gated not in ACTIVATIONS:
         raise KernelError(f"expert_product: unknown activation '{gated}'")
     check(lib().gi_expert_product(_dev(a, "a"), dtype_code(a.dtype), K, int(a_div), _dev(w, "w"), dtype_code(w.dtype), rows * K, K,
-                                  N * K if gated else 0, int(gated is not None), ACTIVATIONS.get(gated, 0), float(limit), _dev(out, "out"),
+                                  N * K if gated else 0, int(gated is not None),
+                                  ACTIVATIONS[gated] if gated else PLAIN_ACTIVATIONS[act or "none"], float(limit), _dev(out, "out"),
                                   dtype_code(out.dtype), N, N, K, _dev(tile_group, "tile_group", torch.int32),
                                   _dev(sorted_rows, "sorted_rows", torch.int32), _dev(n_tiles, "n_tiles", torch.int32),
                                   tile_group.numel(), _stream()), "expert_product")
@@ -682,6 +777,42 @@ def causal_conv(proj: torch.Tensor, offset: int, weight: torch.Tensor, bias: Opt
                                _dev(out, "out", torch.float32), C, taps, T, R, int(bool(activate)), _stream()), "causal_conv")
     if taps > 1:
         count_launches(1)
+
+
+def gated_delta(proj: torch.Tensor, in_offset: int, b_offset: int, a_offset: int, conv: torch.Tensor, a_log: torch.Tensor,
+                dt_bias: torch.Tensor, q_scale: float, state: torch.Tensor, state_offset: int, conv_offset: int,
+                row_req: torch.Tensor, seg_start: torch.Tensor, seg_len: torch.Tensor, state_slots: torch.Tensor, qkv: torch.Tensor,
+                gates: torch.Tensor, out: torch.Tensor, num_heads: int, key_heads: int, dk: int, dv: int,
+                narrow: Optional[bool] = None, unit_eps: float = 1e-6) -> None:
+    """The gated delta rule over each request's rows in order. ``proj`` [T, ld] holds the projections of q, k (key_heads of
+    dk) and v (H heads of dv) side by side from in_offset and those of b and a (H each). q, k and v pass a causal convolution
+    (``conv`` [channels, taps], the last column weighs the token itself; its last taps - 1 inputs are the block [taps - 1,
+    channels] at conv_offset of the request's slot) and SiLU; q and k of a head are divided by sqrt(sum of squares +
+    unit_eps), q multiplied by q_scale; beta = sigmoid(b), g = exp(-exp(a_log) softplus(a + dt_bias)). Then per head (which
+    reads key head h // (H / key_heads)), with the state S [dk, dv] at state_offset of the slot: S <- g S;
+    u = beta (v - S^T k); S <- S + k u^T; ``out``[t, h] = S^T q. ``qkv`` [T, channels] and ``gates`` [T, 2 H] are workspaces.
+    ``narrow``: how a head's columns are spread (see the kernel; chosen by the rows per request when None); results are the
+    same bit for bit. Two launches."""
+    T, ld = proj.shape
+    C, taps = conv.shape
+    if C != 2 * key_heads * dk + num_heads * dv or qkv.shape != (T, C) or gates.shape != (T, 2 * num_heads) or out.shape != (T, num_heads * dv):
+        raise KernelError("gated_delta: shapes do not agree")
+    if a_log.numel() != num_heads or dt_bias.numel() != num_heads:
+        raise KernelError("gated_delta: a_log and dt_bias must have one value per head")
+    if state.dim() != 2 or state_offset < 0 or state_offset + num_heads * dk * dv > state.shape[1] or conv_offset < 0 or \
+            conv_offset + (taps - 1) * C > state.shape[1]:
+        raise KernelError("gated_delta: the state does not fit the slot")
+    R = seg_start.numel()
+    if narrow is None:
+        narrow = T > 4 * R
+    check(lib().gi_gated_delta(
+        _dev(proj, "proj", torch.float32), ld, int(in_offset), int(b_offset), int(a_offset), _dev(conv, "conv", torch.float32), taps,
+        _dev(a_log, "a_log", torch.float32), _dev(dt_bias, "dt_bias", torch.float32), float(q_scale), float(unit_eps),
+        _dev(state, "state", torch.float32), state.shape[1], int(state_offset), int(conv_offset), _dev(row_req, "row_req", torch.int32),
+        _dev(seg_start, "seg_start", torch.int32), _dev(seg_len, "seg_len", torch.int32), _dev(state_slots, "state_slots", torch.int32),
+        _dev(qkv, "qkv", torch.float32), _dev(gates, "gates", torch.float32), _dev(out, "out", torch.float32), T, R, num_heads,
+        key_heads, dk, dv, int(bool(narrow)), _stream()), "gated_delta")
+    count_launches(1)
 
 
 def linear_scan(q: torch.Tensor, q_offset: int, k: torch.Tensor, k_offset: int, v: torch.Tensor, v_offset: int,
@@ -1099,14 +1230,24 @@ AHEAD_BYTES = 24 << 20
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False, plan=None,
-            w_tiles: Optional[torch.Tensor] = None, ahead: Optional[torch.Tensor] = None) -> None:
+            w_tiles: Optional[torch.Tensor] = None, ahead: Optional[torch.Tensor] = None, act: Optional[str] = None) -> None:
     """out[M,N] (+)= a[M,K] @ w[N,K]^T on the tensor cores: bfloat16 operands, 32-bit accumulation,
     output 32-bit (optionally accumulated into) or bfloat16. K must be a multiple of 8. ``w_tiles``
     (tile_weight(w)) lets products of few tokens fetch the weights with bulk copies. ``ahead``: a tensor
     that a later kernel of the step streams (the tile-by-tile weights of the next large product); a product of few
-    tokens asks its first AHEAD_BYTES into L2 while it runs, so that memory keeps streaming between the kernels."""
+    tokens asks its first AHEAD_BYTES into L2 while it runs, so that memory keeps streaming between the kernels.
+    ``act`` (one of PLAIN_ACTIVATIONS, bfloat16 output): applied to the sums before they are rounded."""
     M, K = a.shape
     N = w.shape[0]
+    if act is not None and (act not in PLAIN_ACTIVATIONS or out.dtype is not torch.bfloat16 or accumulate):
+        raise KernelError(f"gemm_tc: activation '{act}' is unknown or the output is not a stored bfloat16 matrix")
+    if act is not None and plan is None and M > 128 and N % 8 == 0:      # many tokens: the activation in the persistent kernel's epilogue
+        st = _tc_state(a.device)
+        block_q = 256 if N >= 256 else 128
+        check(lib().gi_gemm_tc_persistent(_dev(a, "a", torch.bfloat16), _dev(w, "w", torch.bfloat16), _dev(out, "out"),
+                                          4 | (PLAIN_ACTIVATIONS[act] << 8), M, N, K, K, K, N, block_q, st.status.data_ptr(), 1, 0, 0,
+                                          _paired(M, block_q), 0.0, 0, _stream()), "gemm_tc")
+        return
     if w.shape[1] != K or out.shape != (M, N):
         raise KernelError(f"gemm: shapes do not agree (a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)})")
     key = (M, N, K, out.dtype, w_tiles is not None, bool(accumulate)) if plan is None else None
@@ -1140,7 +1281,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: boo
             count_launches(1)     # the kernel that adds the ranges up
         return
     check(lib().gi_gemm_tc(_dev(a, "a", torch.bfloat16), _dev(w, "w", torch.bfloat16), _dev(out, "out"),
-                           dtype_code(out.dtype), int(accumulate), M, N, K, K, K, N, int(swap), block_q, splits,
+                           dtype_code(out.dtype) | (PLAIN_ACTIVATIONS[act] << 8 if act else 0), int(accumulate), M, N, K, K, K, N, int(swap), block_q, splits,
                            st.workspace.data_ptr(), st.workspace.numel(), st.counters.data_ptr(), st.counters.numel(),
                            st.status.data_ptr(), _opt(w_tiles, "w_tiles", torch.bfloat16),
                            ahead.data_ptr() if ahead is not None and swap and M <= 32 else 0,

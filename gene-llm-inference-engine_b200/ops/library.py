@@ -48,7 +48,7 @@ _SIGNATURES = {
                         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_longlong, c_int, c_void_p],
     "gi_expert_product": [c_void_p, c_int, c_longlong, c_int, c_void_p, c_int, c_longlong, c_int, c_longlong, c_int, c_int, c_float,
                           c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
-    "gi_route": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+    "gi_route": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
                  c_void_p, c_int, c_int, c_void_p, c_void_p],
     "gi_gather_rows": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
     "gi_route_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -60,8 +60,17 @@ _SIGNATURES = {
     "gi_sigmoid_gate": [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
     "gi_softcap": [c_void_p, c_longlong, c_float, c_void_p],
     "gi_scale": [c_void_p, c_longlong, c_float, c_void_p],
-    "gi_depth_mix": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_float, c_void_p, c_int,
-                     c_int, c_int, c_void_p],
+    "gi_depth_mix": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float,
+                     c_void_p, c_int, c_int, c_int, c_void_p],
+    "gi_layer_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
+    "gi_plain_act": [c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p],
+    "gi_take_stream": [c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_void_p],
+    "gi_maps_norm_store": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_float, c_void_p, c_void_p,
+                           c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "gi_maps_combine": [c_void_p, c_int, c_void_p, c_int, c_float, c_float, c_float, c_int, c_int, c_int, c_void_p],
+    "gi_gated_delta": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                       c_longlong, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                       c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "gi_streams": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p,
                    c_int, c_int, c_int, c_void_p],
     "gi_grouped_tile_rows": [],

@@ -42,7 +42,16 @@ class AttentionMixer:
     ``conv_taps`` n: every channel of the [q; k; v] projection passes a causal convolution over the request's last n
     tokens before anything else (``conv`` [channels, n], column n-1 weighs the newest token; no bias, no activation;
     nothing before the first token; one tap is a factor per channel); the request's last n-1 projected rows are state, kept
-    in its state slot from ``state_offset`` on."""
+    in its state slot from ``state_offset`` on.
+
+    ``maps`` = 2 (with ``map_weight`` and ``map_factor``): every head has two score maps over the same values. ``num_heads`` and
+    ``num_kv_heads`` count heads, ``head_dim`` is the width of one map; a head's queries and keys are [map 1, map 2] in
+    ``w_qkv`` (2 H hd query rows, 2 Hkv hd key rows), each map brought to unit RMS and weighted on its own (``qk_norm_eps``,
+    ``q_norm`` and ``k_norm`` [hd]). With a1, a2 the maps' attention outputs and w = exp(sum lq1 lk1) - exp(sum lq2 lk2) +
+    map_weight (weights ``lq1``, ``lk1``, ``lq2``, ``lk2`` [hd]), a head's output is map_factor * N(a1 - w a2), N to unit RMS over the
+    value width (eps ``qk_norm_eps``). ``query_temperature`` (coef, every): the queries at position p are multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1). The cache holds [map 1, map 2] in one key row per key head; to the attention
+    kernels these are 2 H query heads ([map 1, 0] and [0, map 2]) over Hkv key heads of 2 hd, which share the rows they read."""
 
     graph_safe = True      # launches depend only on the step's shape: decode steps may be captured in a CUDA graph
 
@@ -56,7 +65,13 @@ class AttentionMixer:
         self.window = params.get("window")
         if self.num_heads % self.num_kv_heads:
             raise ValueError("attention: num_heads must be a multiple of num_kv_heads")
-        if not kernels.attention_supported(self.head_dim):
+        self.maps = int(params.get("maps", 1))
+        self.temperature = None
+        if self.maps not in (1, 2):
+            raise ValueError("attention: heads have one score map or two")
+        if self.maps == 2:
+            self._init_maps(params, weights, build)
+        elif not kernels.attention_supported(self.head_dim):
             raise ValueError(f"attention: head size {self.head_dim} is not supported by the attention kernels "
                              f"(up to 256)")
         pos_spec = params.get("position") or PartSpec("none", {})
@@ -65,7 +80,7 @@ class AttentionMixer:
         if params.get("values", "projected") not in ("projected", "keys"):
             raise ValueError(f"attention: unknown source of values '{params.get('values')}'")
         self.qk_norm_eps = params.get("qk_norm_eps")
-        self.value_dim = int(params.get("value_dim") or self.head_dim)
+        self.value_dim = int(params.get("value_dim") or params["head_dim"])
         self.chunk = params.get("chunk")
         self.learned_sink = params.get("sink") == "learned"
         self.softcap = float(params["softcap"]) if params.get("softcap") else None
@@ -81,6 +96,9 @@ class AttentionMixer:
         # these options are served by the row-form kernel only
         self.row_form = (self.value_dim != self.head_dim or self.chunk is not None or self.learned_sink or
                          self.slopes is not None or self.softcap is not None)
+        if self.maps == 2:        # two maps: the row-form kernel wherever the tensor-core kernels are not built for the sizes
+            self.row_form = self.row_form or build.compute_dtype is not torch.bfloat16 or \
+                not kernels.attention_fast_supported(self.head_dim, self.num_heads, self.num_kv_heads)
         self.sink = bool(params.get("sink", False))
         self.head_gate = bool(params.get("head_gate", False))
         self.out_scale = float(params.get("out_scale", 1.0))
@@ -110,7 +128,9 @@ class AttentionMixer:
         self.cap_only = (self.softcap is not None and self.value_dim == self.head_dim and self.chunk is None and self.slopes is None
                          and not self.learned_sink and not params.get("sink") and build.compute_dtype is torch.bfloat16)
         self.q_norm = self.k_norm = None
-        if self.qk_norm_eps is not None and not params.get("qk_norm_weights", True):
+        if self.maps == 2:
+            self.q_norm, self.k_norm = (_vector_of(weights, n, self.map_dim, build) for n in ("q_norm", "k_norm"))
+        elif self.qk_norm_eps is not None and not params.get("qk_norm_weights", True):
             self.q_norm = self.k_norm = torch.ones(self.head_dim, dtype=torch.float32, device=build.device)
         elif self.qk_norm_eps is not None:
             for name, heads in (("q_norm", self.num_heads), ("k_norm", self.num_kv_heads)):
@@ -120,12 +140,13 @@ class AttentionMixer:
                 setattr(self, name, weights[name].to(device=build.device, dtype=torch.float32).contiguous())
         if self.wide_norm and (self.qk_norm_eps is None or not params.get("qk_norm_weights", True)):
             raise ValueError("attention: qk_norm_wide needs qk_norm_eps and weights")
-        qkv_rows = (self.num_heads + self.num_kv_heads) * self.head_dim + \
+        query_rows = self.num_heads * self.head_dim // self.maps
+        qkv_rows = query_rows + self.num_kv_heads * self.head_dim + \
             (0 if self.values_are_keys else self.num_kv_heads * self.value_dim) + (self.num_heads if self.head_gate else 0)
         if tuple(weights["w_qkv"].shape) != (qkv_rows, self.hidden_size):
             raise ValueError(f"attention: w_qkv has shape {tuple(weights['w_qkv'].shape)}, expected "
                              f"({qkv_rows}, {self.hidden_size})")
-        if tuple(weights["w_o"].shape) != (self.hidden_size, self.num_heads * self.value_dim):
+        if tuple(weights["w_o"].shape) != (self.hidden_size, self.num_heads // self.maps * self.value_dim):
             raise ValueError(f"attention: w_o has shape {tuple(weights['w_o'].shape)}")
         self.conv = None
         if self.conv_taps is not None:
@@ -148,6 +169,30 @@ class AttentionMixer:
         if self.fast or self.cap_fast:
             self.chunk_keys = kernels.attention_chunk_keys()
             self.max_chunks = (build.max_position + self.chunk_keys - 1) // self.chunk_keys
+
+    def _init_maps(self, params, weights, build) -> None:
+        """Heads of two score maps: from here on ``num_heads`` and ``head_dim`` are what the attention kernels see."""
+        for option in ("window", "chunk", "sink", "softcap", "head_gate", "distance_slopes", "conv_taps", "qk_norm_wide"):
+            if params.get(option):
+                raise ValueError(f"attention: '{option}' cannot be combined with two score maps")
+        if params.get("values", "projected") != "projected" or params.get("out_scale", 1.0) != 1.0 or \
+                (params.get("position") is not None and params["position"].kind != "none"):
+            raise ValueError("attention: two score maps take projected values, no output factor and no rotation")
+        if params.get("qk_norm_eps") is None or not params.get("qk_norm_weights", True):
+            raise ValueError("attention: two score maps need qk_norm_eps and weights")
+        self.map_heads, self.map_dim = self.num_heads, self.head_dim
+        self.num_heads, self.head_dim = 2 * self.num_heads, 2 * self.head_dim
+        vd = int(params.get("value_dim") or self.map_dim)
+        if not kernels.attention_rows_supported(self.head_dim, vd) or not kernels.maps_combine_supported(vd):
+            raise ValueError(f"attention: two maps of size {self.map_dim} with value size {vd} are not supported")
+        lq1, lk1, lq2, lk2 = (_vector_of(weights, n, self.map_dim, build).double() for n in ("lq1", "lk1", "lq2", "lk2"))
+        self.map_weight = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + float(params["map_weight"])
+        self.map_factor = float(params["map_factor"])
+        if params.get("query_temperature"):
+            coef, every = (float(v) for v in params["query_temperature"])
+            if not every > 0:
+                raise ValueError("attention: the query temperature's blocks must have a positive length")
+            self.temperature = (coef, every)
 
     def prefill_on_tcgen05(self, page_size: int) -> bool:
         """Head sizes 64 and 128 with pages TMA can tile: prompt portions run on the tcgen05 kernel."""
@@ -275,9 +320,15 @@ class AttentionMixer:
             kernels.causal_conv(proj, 0, self.conv, None, state, self.state_offset if self.conv_taps > 1 else 0, ctx.row_req,
                                 ctx.seg_start, ctx.seg_len, ctx.state_slots, mixed, activate=False)
             proj = mixed
-        k_off = H * hd
+        k_off = H * hd // self.maps
         v_off = k_off if self.values_are_keys else k_off + Hkv * hd
         gate_off = v_off + Hkv * hd
+        if self.maps == 2:
+            kernels.maps_norm_store(proj, 0, k_off, v_off, self.q_norm, self.k_norm, self.qk_norm_eps, self.temperature, ctx.positions,
+                                    ctx.row_req, tables, q, k_cache, v_cache, self.map_heads, Hkv, self.map_dim, self.value_dim,
+                                    ctx.page_size, write_kv=run.writes_cache)
+            self._attend_maps(ctx, q, k_cache, v_cache, tables, x, then)
+            return
         kernels.norm_rope_store(proj, 0, k_off, v_off, self.q_norm, self.k_norm, self.qk_norm_eps or 0.0,
                                 getattr(self.position, "freq", None), self.position.interleaved, ctx.positions,
                                 ctx.row_req, tables, q, k_cache, v_cache, H, Hkv, hd, ctx.page_size,
@@ -307,3 +358,24 @@ class AttentionMixer:
         self._attend(ctx, q, k_cache, v_cache, att, tables, sink=self.sink, gate=proj if self.head_gate else None,
                      gate_offset=gate_off, out_scale=self.out_scale)
         self.w_o.forward(att, x, accumulate=True, then=then)
+
+    def _attend_maps(self, ctx, q, k_cache, v_cache, tables, x, then) -> None:
+        """Both maps of every head in one attention call, then their difference and the output projection."""
+        T, H, vd = q.shape[0], self.num_heads, self.value_dim
+        if self.row_form:
+            both = ctx.scratch("att_maps", (T, H * vd), torch.float32)
+            kernels.attention_rows_of_step(ctx, q, k_cache, v_cache, both, tables, H, self.num_kv_heads, self.head_dim, vd, self.scale,
+                                           None, None, None, None)
+        else:
+            both = ctx.scratch("att_maps", (T, H * vd), self.dtype)
+            self._attend(ctx, q, k_cache, v_cache, both, tables)
+        att = ctx.scratch("att", (T, self.map_heads * vd), self.dtype)
+        kernels.maps_combine(both, att, self.map_weight, self.qk_norm_eps, self.map_factor, self.map_heads)
+        self.w_o.forward(att, x, accumulate=True, then=then)
+
+
+def _vector_of(weights, name: str, n: int, build) -> torch.Tensor:
+    w = weights[name]
+    if tuple(w.shape) != (n,):
+        raise ValueError(f"attention: {name} has shape {tuple(w.shape)}, expected ({n},)")
+    return w.to(device=build.device, dtype=torch.float32).contiguous()

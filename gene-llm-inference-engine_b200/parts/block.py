@@ -3,7 +3,9 @@ from __future__ import annotations
 
 import torch
 
+from .norm import LayerNorm
 from .registry import FEED_FORWARDS, MIXERS, NORMS, build_part, register_block, sub_weights
+from .stream import EmbeddingMix
 
 
 @register_block("pre_norm")
@@ -176,8 +178,9 @@ class ParallelBlock:
 
     The stream stays 32-bit. Both sublayers add into ``y``, which is zero when they start; one kernel then forms fresh
     (adding the bias of the feed-forward's last product, if it has one),
-    keeps it in the step's history [tokens, slots, width], mixes, clears y and, when the next block is of this kind with a
-    norm of a single weight, writes that block's normed input in the same pass (``ctx.carry``)."""
+    keeps it in the step's history [tokens, slots, width], mixes, clears y and writes what runs next reads in the same pass
+    (``ctx.carry``): the normed input of a next block of this kind (a norm of a single weight, or a layer norm), or the stream
+    in the compute dtype when a product over it replaces the stream (``EmbeddingMix``)."""
 
     def __init__(self, layer_spec, weights, build):
         bp = layer_spec.block_params
@@ -202,14 +205,12 @@ class ParallelBlock:
                 raise ValueError(f"parallel block: {w.numel()} depth weights, expected {self.slot + 1}")
             self.depth_weights = w.reshape(-1).to(device=build.device, dtype=torch.float32).contiguous()
         self.dtype = build.compute_dtype
-        self._next = None           # the block of the next run, when this kernel can write its normed input
+        self._next = {}             # run (by the layer whose cache it uses) -> what runs after it, when this kernel can prepare that
 
-    def followed_by(self, block) -> None:
-        ok = isinstance(block, ParallelBlock) and hasattr(block.mixer_norm, "scalar")
-        if self._next is None and ok:
-            self._next = block
-        elif self._next is not block:
-            self._next = False      # several successors (a layer that runs more than once): nothing is prepared
+    def followed_in_run(self, run, after) -> None:
+        ok = isinstance(after, EmbeddingMix) or (isinstance(after, ParallelBlock) and
+                                                 (hasattr(after.mixer_norm, "scalar") or isinstance(after.mixer_norm, LayerNorm)))
+        self._next[run.cache_layer] = after if ok and self._next.get(run.cache_layer, after) is after else None
 
     def forward(self, ctx, run, x: torch.Tensor) -> None:
         from ..ops import kernels
@@ -222,7 +223,9 @@ class ParallelBlock:
         # what the block before left: y = 0 everywhere, xn = this block's normed input, the history filled up to its slot
         ready = state is not None and state[0] == x.data_ptr() and state[1] is self
         first = self.slot and not (state is not None and state[0] == x.data_ptr() and state[2])
-        nxt = self._next if self._next else None
+        nxt = self._next.get(run.cache_layer)
+        if isinstance(nxt, EmbeddingMix) and getattr(ctx, "tapping", False):
+            nxt = None              # someone listens to the stream: it stays in its place
 
         def layer():
             if not ready:
@@ -232,9 +235,14 @@ class ParallelBlock:
             self.mixer.forward(ctx, run, xn, y)
             if self.feed_forward is not None:
                 self.feed_forward.forward(ctx, xn, y)
-            kernels.depth_mix(x, y, self.mult, hist, self.slot, self.depth_weights, first=bool(first),
-                              next_weight=nxt.mixer_norm.scalar if nxt else None, eps=nxt.mixer_norm.eps if nxt else 0.0,
-                              xn_out=xn if nxt else None, y_bias=self.y_bias)
+            after = {}
+            if isinstance(nxt, EmbeddingMix):
+                after = {"handover": nxt.start(ctx), "xn_out": nxt.taken(ctx)}
+            elif nxt is not None and isinstance(nxt.mixer_norm, LayerNorm):
+                after = {"next_weight": nxt.mixer_norm.weight, "next_bias": nxt.mixer_norm.bias, "eps": nxt.mixer_norm.eps, "xn_out": xn}
+            elif nxt is not None:
+                after = {"next_weight": nxt.mixer_norm.scalar, "eps": nxt.mixer_norm.eps, "xn_out": xn}
+            kernels.depth_mix(x, y, self.mult, hist, self.slot, self.depth_weights, first=bool(first), y_bias=self.y_bias, **after)
 
         parts = [(self.mixer_norm, None), (self.mixer, run)] + ([(self.feed_forward, None)] if self.feed_forward is not None else [])
         key = _launch_key(ctx, *parts)
@@ -246,6 +254,8 @@ class ParallelBlock:
         ctx.tap("ffn_out", run.layer, x)
         if carry is not None:
             carry["parallel"] = (x.data_ptr(), nxt, bool(self.slot))
+            if isinstance(nxt, EmbeddingMix):
+                carry["stream_handed"] = (x.data_ptr(), id(nxt))
 
 
 @register_block("hyper_connections")

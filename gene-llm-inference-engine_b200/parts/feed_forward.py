@@ -80,19 +80,64 @@ class SwiGLUFeedForward:
             kernels.add_bias(x, self.b_down)
 
 
+@register_feed_forward("mlp")
+class UngatedFeedForward:
+    """x += W_down act(W_up xn), act applied by the first product's epilogue.
+
+    Params: ``hidden_size``, ``intermediate_size`` and ``activation`` (one of ``kernels.PLAIN_ACTIVATIONS``: "relu2", the square
+    of ReLU). Weights: ``w_up`` [I, hidden], ``w_down`` [hidden, I]."""
+
+    graph_safe = True
+
+    def __init__(self, params, weights, build):
+        self.hidden_size, self.intermediate_size = int(params["hidden_size"]), int(params["intermediate_size"])
+        self.activation = params["activation"]
+        if self.activation not in kernels.PLAIN_ACTIVATIONS:
+            raise ValueError(f"feed-forward: unknown activation '{self.activation}'")
+        I, D = self.intermediate_size, self.hidden_size
+        for name, shape in (("w_up", (I, D)), ("w_down", (D, I))):
+            if tuple(weights[name].shape) != shape:
+                raise ValueError(f"feed-forward: {name} has shape {tuple(weights[name].shape)}, expected {shape}")
+        self.w_up = Linear(weights["w_up"], build.compute_dtype, build.device, tiles=build.weight_tiles)
+        self.w_down = Linear(weights["w_down"], build.compute_dtype, build.device, tiles=build.weight_tiles)
+        self.dtype = build.compute_dtype
+
+    @property
+    def first_product(self):
+        return self.w_up
+
+    def launch_key(self, ctx):
+        return ()
+
+    def forward(self, ctx, xn: torch.Tensor, x: torch.Tensor) -> None:
+        h = ctx.scratch("ffn_hidden", (xn.shape[0], self.intermediate_size), self.dtype)
+        if self.dtype is torch.bfloat16 and self.hidden_size % 8 == 0:
+            kernels.gemm_tc(xn, self.w_up.weight, h, w_tiles=self.w_up.weight_tiles, act=self.activation)
+        else:
+            z = ctx.scratch("ffn_up", (xn.shape[0], self.intermediate_size), torch.float32)
+            self.w_up.forward(xn, z)
+            kernels.plain_act(z, h, self.activation)
+        self.w_down.forward(h, x, accumulate=True)
+
+
 @register_feed_forward("routed_experts")
 class RoutedExpertsFeedForward:
     """A mixture of small gated feed-forwards of which every token uses ``top``: with z = W_r u in 32-bit and
     s = sigmoid(z), the experts with the largest s_e + ``correction``_e are chosen (the correction steers the choice
     only), and x += sum over the chosen e of s_e * W_down,e (act(W_gate,e u) * (W_up,e u)); the weights s_e are used
     as they are, not renormalised. With ``router`` = "table" nothing is scored: row ``token id`` of ``table`` [vocab, top]
-    names the token's experts (different ones), each with weight 1 / top. ``shared``: the params of a gated feed-forward
+    names the token's experts (different ones), each with weight 1 / top. ``shared``: the params of a feed-forward
     that every token runs besides, added to the sum.
+
+    ``scores`` = "softmax": s = softmax(z) over all experts; ``renormalise``: the chosen s_e are divided by their sum
+    (+ 1e-20); ``router_scale``: a constant on the weights. ``gated`` False: an expert is W_down,e act(W_up,e u) with
+    ``activation`` one of ``kernels.PLAIN_ACTIVATIONS`` (and so is the shared one).
 
     Params: ``hidden_size``, ``intermediate_size`` (of one expert), ``experts``, ``top`` and optionally ``activation``
     ("silu") with ``activation_limit``, ``router`` ("scored", the default, or "table", then with ``vocab_size``), ``shared``.
     Weights: ``router`` [E, hidden] and ``correction`` [E] (scored) or ``table`` [vocab, top] integers, ``w_gate_up``
-    [E, 2I, hidden] (an expert's gate rows, then its up rows), ``w_down`` [E, hidden, I], the shared expert's under ``shared.``.
+    [E, 2I, hidden] (an expert's gate rows, then its up rows; not gated: ``w_up`` [E, I, hidden]), ``w_down`` [E, hidden, I],
+    the shared expert's under ``shared.``. The ``correction`` may be absent (no correction).
 
     The step's (token, choice) pairs are bucketed by expert on the device into tiles of rows; each tile runs its
     expert's matrices. Few pairs (decoding) and the 32-bit path: tiles of a few rows on the CUDA cores, the expert
@@ -109,7 +154,8 @@ class RoutedExpertsFeedForward:
         self.hidden_size, self.intermediate_size = int(params["hidden_size"]), int(params["intermediate_size"])
         self.experts, self.top = int(params["experts"]), int(params["top"])
         self.activation = params.get("activation", "silu")
-        if self.activation not in kernels.ACTIVATIONS:
+        self.gated = bool(params.get("gated", True))
+        if self.activation not in (kernels.ACTIVATIONS if self.gated else kernels.PLAIN_ACTIVATIONS):
             raise ValueError(f"routed experts: unknown activation '{self.activation}'")
         if not (1 <= self.top <= self.experts):
             raise ValueError(f"routed experts: top {self.top} must lie between 1 and the {self.experts} experts")
@@ -119,17 +165,24 @@ class RoutedExpertsFeedForward:
         self.routing = params.get("router", "scored")
         if self.routing not in ("scored", "table"):
             raise ValueError(f"routed experts: unknown router '{self.routing}' (known: scored, table)")
+        self.scores = params.get("scores", "sigmoid")
+        if self.scores not in ("sigmoid", "softmax"):
+            raise ValueError(f"routed experts: unknown scores '{self.scores}' (known: sigmoid, softmax)")
+        self.renormalise, self.router_scale = bool(params.get("renormalise", False)), float(params.get("router_scale", 1.0))
         E, I, D = self.experts, self.intermediate_size, self.hidden_size
-        chooser = (("router", (E, D)), ("correction", (E,))) if self.routing == "scored" else \
-            (("table", (int(params["vocab_size"]), self.top)),)
-        for name, shape in chooser + (("w_gate_up", (E, 2 * I, D)), ("w_down", (E, D, I))):
+        chooser = (("router", (E, D)),) if self.routing == "scored" else (("table", (int(params["vocab_size"]), self.top)),)
+        if self.routing == "scored" and "correction" in weights:
+            chooser += (("correction", (E,)),)
+        first = ("w_gate_up", (E, 2 * I, D)) if self.gated else ("w_up", (E, I, D))
+        for name, shape in chooser + (first, ("w_down", (E, D, I))):
             if tuple(weights[name].shape) != shape:
                 raise ValueError(f"routed experts: {name} has shape {tuple(weights[name].shape)}, expected {shape}")
         dev, dt = build.device, build.compute_dtype
         self.router = self.correction = self.table = None
         if self.routing == "scored":
             self.router = weights["router"].to(device=dev, dtype=torch.float32).contiguous()
-            self.correction = weights["correction"].to(device=dev, dtype=torch.float32).contiguous()
+            if "correction" in weights:
+                self.correction = weights["correction"].to(device=dev, dtype=torch.float32).contiguous()
         else:
             table = weights["table"]
             if table.is_floating_point():
@@ -143,8 +196,9 @@ class RoutedExpertsFeedForward:
             self.table = table.to(device=dev, dtype=torch.int32).contiguous()
         self.shared = None
         if params.get("shared"):
-            self.shared = SwiGLUFeedForward(params["shared"], sub_weights(weights, "shared."), build)
-        self.w_gate_up = weights["w_gate_up"].to(device=dev, dtype=dt).contiguous()
+            kind = SwiGLUFeedForward if self.gated else UngatedFeedForward
+            self.shared = kind(params["shared"], sub_weights(weights, "shared."), build)
+        self.w_first = weights[first[0]].to(device=dev, dtype=dt).contiguous()
         self.w_down = weights["w_down"].to(device=dev, dtype=dt).contiguous()
         self.dtype = dt
 
@@ -168,8 +222,7 @@ class RoutedExpertsFeedForward:
         n_tiles = ctx.scratch("route_n_tiles", (1,), torch.int32, capacity=1)
         self._route(ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles)
         hidden = ctx.scratch("expert_hidden", (T * top, I), torch.float32, capacity=max(most, T) * top)
-        kernels.expert_product(xn, top, self.w_gate_up, hidden, sorted_rows, tile_group, n_tiles, gated=self.activation,
-                               limit=self.limit)
+        kernels.expert_product(xn, top, self.w_first, hidden, sorted_rows, tile_group, n_tiles, **self._first_form())
         part = ctx.scratch("expert_out", (T * top, D), torch.float32, capacity=max(most, T) * top)
         kernels.expert_product(hidden, 1, self.w_down, part, sorted_rows, tile_group, n_tiles)
         kernels.route_combine(part, weights, x)
@@ -182,7 +235,12 @@ class RoutedExpertsFeedForward:
             kernels.route_table(ctx.tokens, ctx.feedback, self.table, self.experts, ids, weights, sorted_rows, tile_group, n_tiles,
                                 **tiles)
         else:
-            kernels.route(xn, self.router, self.correction, self.top, ids, weights, sorted_rows, tile_group, n_tiles, **tiles)
+            kernels.route(xn, self.router, self.correction, self.top, ids, weights, sorted_rows, tile_group, n_tiles,
+                          scores=self.scores, renormalise=self.renormalise, factor=self.router_scale, **tiles)
+
+    def _first_form(self) -> dict:
+        """What the experts' first product does besides multiplying."""
+        return {"gated": self.activation, "limit": self.limit} if self.gated else {"act": self.activation}
 
     def _forward_tensor_cores(self, ctx, xn: torch.Tensor, x: torch.Tensor, most: int) -> None:
         T = xn.shape[0]
@@ -199,7 +257,7 @@ class RoutedExpertsFeedForward:
         rows = ctx.scratch("expert_rows", (tiles * tm, D), self.dtype, capacity=most_tiles * tm)
         kernels.gather_rows(xn, top, sorted_rows, n_tiles, tm, rows)
         hidden = ctx.scratch("expert_hidden_tc", (tiles * tm, I), self.dtype, capacity=most_tiles * tm)
-        kernels.expert_product_tc(rows, self.w_gate_up, hidden, tile_group, n_tiles, gated=self.activation, limit=self.limit)
+        kernels.expert_product_tc(rows, self.w_first, hidden, tile_group, n_tiles, **self._first_form())
         part = ctx.scratch("expert_out_tc", (tiles * tm, D), torch.float32, capacity=most_tiles * tm)
         kernels.expert_product_tc(hidden, self.w_down, part, tile_group, n_tiles)
         kernels.route_combine(part, weights, x, pair_row=pair_row)

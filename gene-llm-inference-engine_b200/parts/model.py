@@ -14,7 +14,7 @@ import torch
 from ..config import ModelSpec
 from ..ops import kernels
 from ..ops.linear import Linear
-from .registry import BLOCKS, LOGIT_TRANSFORMS, NORMS, POSITION_ENCODINGS, BuildContext, build_part, sub_weights
+from .registry import BLOCKS, LOGIT_TRANSFORMS, NORMS, POSITION_ENCODINGS, STREAM_INPUTS, BuildContext, build_part, sub_weights
 
 
 @dataclass(frozen=True)
@@ -22,6 +22,7 @@ class LayerRun:
     layer: int          # which layer's parts and weights run
     cache_layer: int    # the layer whose pages / state this run uses
     writes_cache: bool
+    stream_input: bool = False      # the stream is replaced (``DecoderModel.stream_input``) right before this run
 
 
 class DecoderModel:
@@ -63,17 +64,20 @@ class DecoderModel:
             self.layers.append(BLOCKS[layer_spec.block](layer_spec, sub_weights(params, f"layers.{i}."), build))
         for i, j in spec.shared_layers.items():
             self.layers[i] = self.layers[j]
-        self.runs = [LayerRun(e.layer, e.layer if e.cache_of is None else e.cache_of, e.writes_cache)
+        self.runs = [LayerRun(e.layer, e.layer if e.cache_of is None else e.cache_of, e.writes_cache, e.stream_input)
                      for e in spec.schedule]
+        # what replaces the stream ahead of the runs that say so; most designs: nothing
+        self.stream_input = None
+        if spec.stream_input is not None:
+            self.stream_input = build_part(STREAM_INPUTS, "stream input", spec.stream_input,
+                                           sub_weights(params, "stream_input."), build)
         self.final_norm = build_part(NORMS, "norm", spec.final_norm, sub_weights(params, "final_norm."), build)
-        # a block may prepare what the block of the next run reads (its normed input): it is told who follows
+        # a block may prepare what the block of the next run (or the stream input ahead of it) reads: it is told, run by run,
+        # who follows
         for run, after in zip(self.runs, self.runs[1:]):
-            follows = getattr(self.layers[run.layer], "followed_by", None)
+            follows = getattr(self.layers[run.layer], "followed_in_run", None)
             if follows is not None:
-                follows(self.layers[after.layer])
-            follows = getattr(self.layers[run.layer], "followed_in_run", None)      # for a layer that runs more than once
-            if follows is not None:
-                follows(run, self.layers[after.layer])
+                follows(run, self.stream_input if after.stream_input else self.layers[after.layer])
         if spec.tie_word_embeddings:
             self.head = Linear.over(self.embedding, tiles=weight_tiles)   # the table itself, not a second row-major copy
         else:
@@ -129,6 +133,7 @@ class DecoderModel:
         visit(self.embedding)
         visit(self.embedding_position)
         visit(self.layers)
+        visit(self.stream_input)
         visit(self.final_norm)
         visit(self.head)
         visit(self.logit_transform)
@@ -147,7 +152,13 @@ class DecoderModel:
             if self.embedding_position is not None:
                 self.embedding_position.add_to(ctx, x)
         ctx.tap("embedding", -1, x)
+        if self.stream_input is not None:
+            with ctx.range("stream input"):
+                self.stream_input.begin(ctx, x)
         for run in self.runs:
+            if run.stream_input:
+                with ctx.range("stream input"):
+                    self.stream_input.forward(ctx, x)
             with ctx.range(f"layer {run.layer}"):
                 self.layers[run.layer].forward(ctx, run, x)
         k = ctx.n_logit_rows

@@ -52,3 +52,26 @@ class ScalarRMSNorm(RMSNorm):
         size = int(params["size"])
         super().__init__(params, {"weight": g.reshape(1).float().expand(size)}, build)
         self.scalar = g.reshape(1).to(device=build.device, dtype=torch.float32).contiguous()
+
+
+@register_norm("layernorm")
+class LayerNorm:
+    """out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight + bias, computed in 32-bit from the 32-bit residual stream.
+    Params: ``size``, ``eps``. Weights: ``weight`` and ``bias`` [size]."""
+
+    def __init__(self, params, weights, build):
+        self.size = int(params["size"])
+        self.eps = float(params["eps"])
+        for name in ("weight", "bias"):
+            w = weights[name]
+            if tuple(w.shape) != (self.size,):
+                raise ValueError(f"layernorm: {name} has shape {tuple(w.shape)}, expected ({self.size},)")
+            setattr(self, name, w.to(device=build.device, dtype=torch.float32).contiguous())
+
+    def launch_key(self, ctx):
+        """Its one launch depends on the number of rows only (which the caller's key holds)."""
+        return ()
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        kernels.layer_norm(x, self.weight, self.bias, out, self.eps, rows)
+        return out

@@ -263,6 +263,83 @@ class GatedLinearAttentionMixer:
         self.w_o.forward(y, x, accumulate=True, then=then)
 
 
+@register_mixer("gated_delta")
+class GatedDeltaMixer:
+    """The gated delta rule: a memory per head that is corrected towards the token's value where the token's key reads it.
+    With u the input row: q, k (``num_key_heads`` heads of dk) and v (H heads of dv) are projections that each pass a
+    causal convolution over the request's last ``conv_taps`` tokens per channel (no bias; nothing before the first token)
+    and SiLU; q and k of a head become unit vectors, x / sqrt(sum x^2 + 1e-6), q times ``query_scale``; head h reads key
+    head h // (H / num_key_heads); beta = sigmoid(W_b u), g = exp(-exp(``a_log``_h) softplus(W_a u + ``dt_bias``_h)) per head.
+    S <- g S; w = beta (v - S^T k); S <- S + k (x) w; y = S^T q: the read-out sees the token's own write.
+    Each head's y is brought to unit RMS over its dv values, weighted by ``norm`` [dv] (one weight for all heads), all heads
+    side by side are multiplied by SiLU(W_g u) and sent through ``w_o``. Everything behind the products is 32-bit. A
+    request's state slot holds S and, behind it, the convolution's last taps-1 inputs [taps-1, channels].
+
+    Params: ``hidden_size``, ``num_heads`` (H), ``num_key_heads``, ``key_dim``, ``value_dim``, ``conv_taps``, ``norm_eps`` and
+    optionally ``query_scale`` (key_dim^-0.5) and ``out_scale``. Weights: ``w_in`` [(2 G dk + 2 H dv + 2 H), hidden] (rows of Wq,
+    Wk, Wv, Wg, Wb, Wa in this order), ``conv`` [2 G dk + H dv, taps] (the last column weighs the token itself), ``a_log`` and
+    ``dt_bias`` [H], ``norm`` [dv], ``w_o`` [hidden, H dv]."""
+
+    graph_safe = True
+    takes_then = True
+
+    def __init__(self, params, weights, build):
+        self.hidden_size = int(params["hidden_size"])
+        self.num_heads, self.key_heads = int(params["num_heads"]), int(params["num_key_heads"])
+        self.dk, self.dv, self.taps = int(params["key_dim"]), int(params["value_dim"]), int(params["conv_taps"])
+        self.eps = float(params["norm_eps"])
+        self.q_scale = float(params.get("query_scale", self.dk ** -0.5))
+        self.out_scale = float(params.get("out_scale", 1.0))
+        H, G, dk, dv, D = self.num_heads, self.key_heads, self.dk, self.dv, self.hidden_size
+        if H % G:
+            raise ValueError("gated delta: num_heads must be a multiple of num_key_heads")
+        if dk > 256:
+            raise ValueError(f"gated delta: key size {dk} exceeds what the recurrence kernel holds (256)")
+        if not (1 <= self.taps <= 17):
+            raise ValueError(f"gated delta: {self.taps} convolution taps are not supported (1 to 17)")
+        self.channels = 2 * G * dk + H * dv
+        rows = self.channels + H * dv + 2 * H
+        for name, shape in (("w_in", (rows, D)), ("conv", (self.channels, self.taps)), ("w_o", (D, H * dv))):
+            if tuple(weights[name].shape) != shape:
+                raise ValueError(f"gated delta: {name} has shape {tuple(weights[name].shape)}, expected {shape}")
+        w_in = weights["w_in"]
+        if rows % 8:              # rows of zeros up to a multiple of 8: the product's output rows then start on 16 bytes
+            w_in = torch.cat([w_in, torch.zeros(8 - rows % 8, D, dtype=w_in.dtype, device=w_in.device)])
+        self.w_in = Linear(w_in, build.compute_dtype, build.device, tiles=build.weight_tiles)
+        self.w_o = Linear(weights["w_o"], build.compute_dtype, build.device, tiles=build.weight_tiles)
+        self.conv = weights["conv"].to(device=build.device, dtype=torch.float32).contiguous()
+        self.a_log = _vector(weights, "a_log", H, build, "gated delta")
+        self.dt_bias = _vector(weights, "dt_bias", H, build, "gated delta")
+        self.norm = _vector(weights, "norm", dv, build, "gated delta").repeat(H).contiguous()
+        self.dtype = build.compute_dtype
+        self.state_offset = 0
+
+    def cache_need(self):
+        return None
+
+    def state_need(self):
+        return StateNeed((self.num_heads * self.dk * self.dv + (self.taps - 1) * self.channels,), "float32")
+
+    def launch_key(self, ctx, run):
+        return (run.cache_layer, ctx.n_requests)
+
+    def forward(self, ctx, run, xn: torch.Tensor, x: torch.Tensor, then=None) -> None:
+        T = xn.shape[0]
+        H, dk, dv, C = self.num_heads, self.dk, self.dv, self.channels
+        proj = ctx.scratch("delta_proj", (T, self.w_in.out_features), torch.float32)
+        self.w_in.forward(xn, proj)
+        qkv = ctx.scratch("delta_qkv", (T, C), torch.float32)
+        gates = ctx.scratch("delta_gates", (T, 2 * H), torch.float32)
+        o = ctx.scratch("delta_out", (T, H * dv), torch.float32)
+        b = C + H * dv
+        kernels.gated_delta(proj, 0, b, b + H, self.conv, self.a_log, self.dt_bias, self.q_scale, ctx.state(run.cache_layer),
+                            self.state_offset, self.state_offset + H * dk * dv, ctx.row_req, ctx.seg_start, ctx.seg_len,
+                            ctx.state_slots, qkv, gates, o, H, self.key_heads, dk, dv)
+        y = ctx.scratch("delta_normed", (T, H * dv), self.dtype)
+        kernels.gated_group_norm(o, proj, C, self.norm, y, H, self.eps, gate_first=False, gate_act="silu", out_scale=self.out_scale)
+        self.w_o.forward(y, x, accumulate=True, then=then)
+
+
 @register_mixer("parallel")
 class ParallelMixer:
     """Several mixers side by side on the same input. ``combine`` "sum" (the default): x += sum_i scale_i * mixer_i(xn).

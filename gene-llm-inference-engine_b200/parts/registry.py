@@ -18,6 +18,7 @@ NORMS: Dict[str, Callable] = {}
 POSITION_ENCODINGS: Dict[str, Callable] = {}
 BLOCKS: Dict[str, Callable] = {}
 LOGIT_TRANSFORMS: Dict[str, Callable] = {}     # what an architecture does to its logits after the head; none is built in
+STREAM_INPUTS: Dict[str, Callable] = {}        # what replaces the residual stream ahead of a run of the schedule that says so
 
 
 @dataclass
@@ -57,6 +58,10 @@ def register_block(kind: str):
 
 def register_logit_transform(kind: str):
     return _register(LOGIT_TRANSFORMS, kind)
+
+
+def register_stream_input(kind: str):
+    return _register(STREAM_INPUTS, kind)
 
 
 def build_part(table: Dict[str, Callable], what: str, spec, weights, build: BuildContext):

@@ -365,6 +365,78 @@ def fovezen_weight_plan(cfg) -> WeightPlan:
     return WeightPlan(rules, [], assemble)
 
 
+def mimolix_weight_plan(cfg) -> WeightPlan:
+    """Tensor names and shapes of a Mimolix checkpoint: ``embed``, ``head``, ``final.norm`` with ``final.norm.b``, ``loop.in`` (when
+    layers are run in passes) and, for layer i, ``l<i>.norm1`` with ``l<i>.norm1.b``, the mixer's tensors under ``l<i>.mix.`` and
+    the feed-forward's under ``l<i>.mlp.`` (``e<k>.up`` / ``.down`` per expert, ``router``, ``shared.up`` / ``.down``). Projections
+    that read the same input become one product: [q; k; v] of the attention, [q; k; v; g; b; a] of the delta mixer, whose
+    three convolutions likewise become one; the experts' matrices are stacked."""
+    D, V = cfg.width, cfg.vocab
+    shift = (0.0, 0.05)                  # the layer norms' biases
+    rules = [TensorRule("embed", (V, D)), TensorRule("head", (V, D)), TensorRule("final.norm", (D,), "vector"),
+             TensorRule("final.norm.b", (D,), "vector", shift)]
+    if cfg.loop is not None:
+        rules.append(TensorRule("loop.in", (D, 2 * D)))
+    for i, layer in enumerate(cfg.layers):
+        p, m = f"l{i}.", layer.mixer
+        rules += [TensorRule(p + "norm1", (D,), "vector"), TensorRule(p + "norm1.b", (D,), "vector", shift)]
+        q = p + "mix."
+        if layer.type == "attention":
+            rules += [TensorRule(q + "q", (2 * m.heads * m.dim, D)), TensorRule(q + "k", (2 * m.kv_heads * m.dim, D)),
+                      TensorRule(q + "v", (m.kv_heads * m.vdim, D)), TensorRule(q + "q.norm", (m.dim,), "vector"),
+                      TensorRule(q + "k.norm", (m.dim,), "vector"), TensorRule(q + "o", (D, m.heads * m.vdim))]
+            rules += [TensorRule(q + n, (m.dim,), "vector", (0.0, 0.1)) for n in ("lq1", "lk1", "lq2", "lk2")]
+        else:
+            for name, rows in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.heads * m.vdim)):
+                rules += [TensorRule(q + name, (rows, D)), TensorRule(q + name + ".conv", (rows, m.conv), "vector", (0.0, 0.5))]
+            rules += [TensorRule(q + "b", (m.heads, D)), TensorRule(q + "a", (m.heads, D)),
+                      TensorRule(q + "A_log", (m.heads,), "vector", ("uniform", -1.5, 1.0)),
+                      TensorRule(q + "dt_bias", (m.heads,), "vector", ("uniform", -4.0, 0.0)),
+                      TensorRule(q + "g", (m.heads * m.vdim, D)), TensorRule(q + "norm", (m.vdim,), "vector"),
+                      TensorRule(q + "o", (D, m.heads * m.vdim))]
+        f = layer.mlp
+        if f is None:
+            continue
+        q = p + "mlp."
+        for e in range(f.experts):
+            rules += [TensorRule(f"{q}e{e}.up", (f.ff, D)), TensorRule(f"{q}e{e}.down", (D, f.ff))]
+        rules.append(TensorRule(q + "router", (f.experts, D)))
+        if f.shared_ff is not None:
+            rules += [TensorRule(q + "shared.up", (f.shared_ff, D)), TensorRule(q + "shared.down", (D, f.shared_ff))]
+
+    def assemble(t: Dict[str, torch.Tensor]) -> Dict[str, torch.Tensor]:
+        out: Dict[str, torch.Tensor] = {"embedding.weight": t["embed"], "head.weight": t["head"], "final_norm.weight": t["final.norm"],
+                                        "final_norm.bias": t["final.norm.b"]}
+        if cfg.loop is not None:
+            out["stream_input.weight"] = t["loop.in"]
+        for i, layer in enumerate(cfg.layers):
+            p, q = f"l{i}.", f"layers.{i}."
+            out[q + "mixer_norm.weight"], out[q + "mixer_norm.bias"] = t[p + "norm1"], t[p + "norm1.b"]
+            a, b = p + "mix.", q + "mixer."
+            if layer.type == "attention":
+                out[b + "w_qkv"] = _cat([t[a + "q"], t[a + "k"], t[a + "v"]])
+                out[b + "q_norm"], out[b + "k_norm"] = t[a + "q.norm"], t[a + "k.norm"]
+                for n in ("lq1", "lk1", "lq2", "lk2"):
+                    out[b + n] = t[a + n]
+            else:
+                out[b + "w_in"] = _cat([t[a + n] for n in ("q", "k", "v", "g", "b", "a")])
+                out[b + "conv"] = _cat([t[a + n + ".conv"] for n in ("q", "k", "v")])
+                out[b + "a_log"], out[b + "dt_bias"], out[b + "norm"] = t[a + "A_log"], t[a + "dt_bias"], t[a + "norm"]
+            out[b + "w_o"] = t[a + "o"]
+            f = layer.mlp
+            if f is None:
+                continue
+            a, b = p + "mlp.", q + "feed_forward."
+            out[b + "w_up"] = torch.stack([t[f"{a}e{e}.up"] for e in range(f.experts)])
+            out[b + "w_down"] = torch.stack([t[f"{a}e{e}.down"] for e in range(f.experts)])
+            out[b + "router"] = t[a + "router"]
+            if f.shared_ff is not None:
+                out[b + "shared.w_up"], out[b + "shared.w_down"] = t[a + "shared.up"], t[a + "shared.down"]
+        return out
+
+    return WeightPlan(rules, [], assemble)
+
+
 def _cat(parts: List[torch.Tensor]) -> torch.Tensor:
     """Concatenates rows; parts of different stored dtypes are widened to 32-bit first."""
     if len({p.dtype for p in parts}) > 1:
