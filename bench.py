@@ -8,6 +8,7 @@
     python bench.py --scenario nipadra               (the Nipadra design beside Llama at equal layer sizes, see run_nipadra)
     python bench.py --scenario gekupel               (the Gekupel design beside Llama at equal layer sizes, see run_gekupel)
     python bench.py --scenario pinorax               (the Pinorax design beside Gekupel and Llama at equal layer sizes, see run_pinorax)
+    python bench.py --scenario mimolix               (the Mimolix design beside Pinorax, Fovezen and Llama at equal layer sizes, see run_mimolix)
     python bench.py --scenario fovezen               (the Fovezen design beside Nipadra and Llama at equal layer sizes, see run_fovezen)
 
 Prints ONE JSON line. ``value`` is decoded tokens per second at batch 8 and context 8192, timed on
@@ -1222,6 +1223,219 @@ def run_fovezen(args):
     return 0
 
 
+# ---------------------------------------------------------------------------------------------- Mimolix beside Pinorax and Fovezen
+def mimolix_config(width, ff, layers, vocab, heads, head_dim):
+    """A Mimolix model with the layer sizes of a Llama shape. Layers in turn: the gated delta rule (width / 128 heads of 128 x 128
+    over half as many key heads, four taps), attention with two score maps (half of Llama's heads, maps of half their head
+    size over values of it, over a quarter as many key heads), the delta rule twice; every layer with the mixture of
+    ``pinorax_config`` (8 experts of which a token uses 2, and a shared one) sized for ungated experts: 9/16 and 3/8 of the
+    dense width, together the dense gated layer's multiply-adds per token. One pass, with the embedding mixed in ahead of it."""
+    moe = {"expert": {"ff": 9 * ff // 16}, "kind": "moe", "router": {"experts": 8, "scale": 2.0, "top": 2}, "shared": {"ff": 3 * ff // 8}}
+    delta = {"conv": 4, "dim": 128, "heads": width // 128, "kv_heads": max(width // 256, 1), "vdim": 128}
+    att = {"diff": 0.5, "dim": head_dim // 2, "heads": heads // 2, "kv_heads": max(heads // 8, 1), "q_temp": {"coef": 0.2, "every": 4096},
+           "scale": (head_dim // 2) ** -0.5, "vdim": head_dim}
+    kinds = [("delta", delta), ("attention", att), ("delta", delta), ("delta", delta)]
+    return {"architecture": "Mimolix", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": 3.0}, "residual_mult": 0.5,
+            "loop": {"start": 0, "stop": layers, "times": 1},
+            "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": moe} for i in range(layers)]}
+
+
+def mimolix_kernel_table(width, ff, heads, head_dim, T, pk):
+    """Each kernel that the Mimolix design added or changed, alone, beside the like kernel of the Fovezen, Pinorax or Gekupel
+    path, at the sizes of one layer: a prompt portion of ``T`` tokens of one request and a decode step of 8 requests at a
+    context of ``T``. ``frac`` is the time the kernel's algorithmic bytes (or, where larger, its multiply-adds on the tensor
+    cores) need at the measured peaks, divided by the time it took; ``frac_of_32bit_issue`` the same against the CUDA cores'
+    32-bit rate, for kernels whose arithmetic has to stay 32-bit."""
+    import torch
+    from geneinfer_b200.ops import kernels as K
+    from geneinfer_b200.ops.linear import Linear
+    dev = torch.device("cuda:0")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rows = []
+    props = torch.cuda.get_device_properties(dev)
+    simt_ops = props.multi_processor_count * 128 * 1.965e9
+    bf = torch.bfloat16
+
+    def add(name, like, fn, nbytes, flops=0.0, simt=0.0):
+        ms = time_calls(fn, flush=flush)
+        ideal = max(nbytes / (pk["hbm_gbs"] * 1e9), flops / (pk["bf16_tflops"] * 1e12)) * 1e3
+        row = {"kernel": name, "like": like, "us": round(ms * 1e3, 1), "frac": round(ideal / ms, 3)}
+        if simt:
+            row["frac_of_32bit_issue"] = round(simt / simt_ops * 1e3 / ms, 3)
+        rows.append(row)
+
+    D, page = width, 16
+    for what, R, n in (("prefill", 1, T), ("decode", 8, 1)):
+        N = R * n
+        i32 = dict(dtype=torch.int32, device=dev)
+        s0, sl, slots = torch.arange(R, **i32) * n, torch.full((R,), n, **i32), torch.arange(R, **i32)
+        rr = torch.arange(R, **i32).repeat_interleave(n)
+        # ends of layers
+        x, y, start = (torch.randn(N, D, device=dev) for _ in range(3))
+        xn = torch.empty(N, D, dtype=bf, device=dev)
+        w, b, one = torch.ones(D, device=dev), torch.zeros(D, device=dev), torch.ones(1, device=dev)
+        add(f"depth_mix with the next layer norm ({what})", "depth_mix", lambda: K.depth_mix(x, y, 0.5, next_weight=w, next_bias=b, eps=1e-6, xn_out=xn), N * D * 18)
+        add(f"depth_mix with the hand-over to a product ({what})", "depth_mix", lambda: K.depth_mix(x, y, 0.5, handover=start, xn_out=xn), N * D * 22)
+        add(f"depth_mix with the next scalar norm, Pinorax ({what})", "", lambda: K.depth_mix(x, y, 0.5, next_weight=one, eps=1e-6, xn_out=xn), N * D * 18)
+        add(f"layer_norm ({what})", "rmsnorm", lambda: K.layer_norm(x, w, b, xn, 1e-6), N * D * 6)
+        add(f"rmsnorm, Llama ({what})", "", lambda: K.rmsnorm(x, w, xn, 1e-6), N * D * 6)
+        # the delta rule, and the linear recurrences of the other designs on states of the same size
+        H, G, dk, dv = D // 128, D // 256, 128, 128
+        C = 2 * G * dk + H * dv
+        proj = torch.randn(N, C + H * dv + 2 * H, device=dev) * 0.5
+        conv = torch.randn(C, 4, device=dev) * 0.3
+        a_log, dt_bias = torch.zeros(H, device=dev), torch.full((H,), -3.0, device=dev)
+        state = torch.zeros(R, H * dk * dv + 3 * C, device=dev)
+        qkv, gates, out = torch.empty(N, C, device=dev), torch.empty(N, 2 * H, device=dev), torch.empty(N, H * dv, device=dev)
+        step_bytes = N * (2 * C + C + H * dv) * 4 + 2 * R * (H * dk * dv + 3 * C) * 4
+        add(f"gated_delta: convolution, unit norms, gates, recurrence ({what})", "linear_scan", lambda: K.gated_delta(
+            proj, 0, C + H * dv, C + H * dv + H, conv, a_log, dt_bias, 0.09, state, 0, H * dk * dv, rr, s0, sl, slots, qkv, gates, out, H, G, dk, dv),
+            step_bytes, simt=N * H * dk * dv * 4.0)
+        cproj = torch.randn(N, C, device=dev)
+        mixed = torch.empty(N, C, device=dev)
+        cst = torch.zeros(R, 3 * C, device=dev)
+        add(f"causal_conv with SiLU, Fovezen ({what})", "", lambda: K.causal_conv(cproj, 0, conv, None, cst, 0, rr, s0, sl, slots, mixed), N * C * 8)
+        lin = torch.randn(N, 2 * H * dk + H * dv, device=dev) * 0.5
+        z, zb = torch.randn(N, H * dk, device=dev) + 3.0, torch.zeros(H * dk, device=dev)
+        parts = {}
+        if N > K.SCAN_PART:
+            parts = {"part_len": K.SCAN_PART, "ws_state": torch.empty(K.scan_parts(N, R), H * dk * dv, device=dev), "ws_decay": torch.empty(N, H * dk, device=dev)}
+        add(f"linear_scan, a decay per row, Fovezen ({what})", "", lambda: K.linear_scan(
+            lin, 0, lin, H * dk, lin, 2 * H * dk, H, 1, dk, dv, False, state, 0, s0, sl, slots, out, row_gate=z, row_gate_bias=zb, tau=16.0,
+            q_scale=0.09, **parts), N * (3 * H * dk + 2 * H * dv) * 4 + 2 * R * H * dk * dv * 4, simt=N * H * dk * dv * (4.0 if parts else 3.0))
+        yb, nw = torch.empty(N, H * dv, dtype=bf, device=dev), torch.ones(H * dv, device=dev)
+        add(f"gated_group_norm per head, SiLU gate after ({what})", "", lambda: K.gated_group_norm(out, proj, C, nw, yb, H, 1e-6, False, gate_act="silu"),
+            N * H * dv * 10)
+        # attention with two maps: projections to pages, attention, difference
+        AH, AG, dim, vd = heads // 2, max(heads // 8, 1), head_dim // 2, head_dim
+        ld = 2 * (AH + AG) * dim + AG * vd
+        aproj = torch.randn(N, ld, device=dev)
+        n_pages = R * ((T + page - 1) // page)
+        kc, vc = (torch.randn(n_pages, AG, page, head_dim, device=dev).to(bf) for _ in range(2))
+        tables = torch.arange(n_pages, **i32).view(R, -1)
+        pos = (torch.arange(n, **i32) + (T - n)).repeat(R)
+        q = torch.empty(N, 4 * AH * dim, dtype=bf, device=dev)
+        hw = torch.ones(dim, device=dev)
+        add(f"maps_norm_store ({what})", "norm_rope_store", lambda: K.maps_norm_store(
+            aproj, 0, 2 * AH * dim, 2 * (AH + AG) * dim, hw, hw, 1e-6, (0.2, 4096), pos, rr, tables, q, kc, vc, AH, AG, dim, vd, page),
+            N * (ld * 4 + (4 * AH * dim + 2 * AG * dim + AG * vd) * 2))
+        # Fovezen's form at as many stored values: heads of the same width, no second map
+        nproj = torch.randn(N, (2 * AH + 2 * AG) * head_dim, device=dev)
+        nq, hw2 = torch.empty(N, 2 * AH * head_dim, dtype=bf, device=dev), torch.ones(head_dim, device=dev)
+        add(f"norm_rope_store, norm per head, no rotation, Fovezen ({what})", "", lambda: K.norm_rope_store(
+            nproj, 0, 2 * AH * head_dim, (2 * AH + AG) * head_dim, hw2, hw2, 1e-6, None, False, pos, rr, tables, nq, kc, vc, 2 * AH, AG, head_dim,
+            page), N * ((2 * AH + 2 * AG) * head_dim * 6))
+        both, att = torch.empty(N, 2 * AH * vd, dtype=bf, device=dev), torch.empty(N, AH * vd, dtype=bf, device=dev)
+        seen = sum(p + 1 for p in range(T - n, T))
+        cache_bytes = R * T * AG * head_dim * 4
+
+        rows_dec = torch.arange(R, **i32)
+        per_tile = 128 // (2 * AH // AG)
+        work = torch.tensor([(t, min(per_tile, n - t), 0) for t in range(0, n, per_tile)][::-1], **i32)
+        chunk = K.attention_chunk_keys()
+        n_chunks = (T + chunk - 1) // chunk
+        part_o, part_ml = torch.empty(R, 2 * AH * n_chunks * head_dim, device=dev), torch.empty(R, 2 * AH * n_chunks * 2, device=dev)
+
+        def attend(out_, nh):
+            if n == 1:
+                K.attention_decode(q, kc, vc, out_, rows_dec, rr, pos, tables, nh, AG, head_dim, page, 0.1, None, part_o, part_ml, n_chunks, n_chunks)
+            else:
+                K.attention_prefill_tc(q, kc, vc, out_, work, pos, tables, nh, AG, head_dim, page, 0.1, None)
+        add(f"attention, two maps ({what})", "attention", lambda: attend(both, 2 * AH), cache_bytes + N * 2 * AH * vd * 4,
+            R * seen * AH * 2.0 * (2 * dim + 2 * vd))
+        add(f"attention, plain heads, Fovezen ({what})", "", lambda: attend(both, 2 * AH), cache_bytes + N * 2 * AH * vd * 4,
+            R * seen * 2 * AH * 4.0 * head_dim)
+        add(f"maps_combine ({what})", "gated_group_norm", lambda: K.maps_combine(both, att, 0.5, 1e-6, 0.5, AH), N * AH * vd * 6)
+        # routing and experts
+        E, top = 8, 2
+        xb = torch.randn(N, D, device=dev).to(bf)
+        router, corr = torch.randn(E, D, device=dev) * 0.02, torch.zeros(E, device=dev)
+        tc_form = N * top >= 256
+        tm = 128 if tc_form else K.grouped_tile_rows()
+        tiles = K.route_tiles(N, top, E, tm)
+        ids, wts = torch.empty(N, top, **i32), torch.empty(N, top, device=dev)
+        srt, grp, cnt, prow = torch.empty(tiles * tm, **i32), torch.empty(tiles, **i32), torch.empty(1, **i32), torch.empty(N * top, **i32)
+        add(f"route + bucket, softmax ({what})", "route", lambda: K.route(xb, router, None, top, ids, wts, srt, grp, cnt, tile_rows=tm, pair_row=prow,
+                                                                         scores="softmax", renormalise=True, factor=2.0), N * D * 2 + E * D * 4)
+        add(f"route + bucket, sigmoid, Gekupel ({what})", "", lambda: K.route(xb, router, corr, top, ids, wts, srt, grp, cnt, tile_rows=tm, pair_row=prow),
+            N * D * 2 + E * D * 4)
+        I, Ig = 9 * ff // 16, 3 * ff // 8
+        wu, wg = torch.randn(E, I, D, device=dev).to(bf) * 0.02, torch.randn(E, 2 * Ig, D, device=dev).to(bf) * 0.02
+        used = min(E, N * top)
+        if tc_form:
+            ar = torch.randn(tiles * tm, D, device=dev).to(bf)
+            h1, h2 = torch.empty(tiles * tm, I, dtype=bf, device=dev), torch.empty(tiles * tm, Ig, dtype=bf, device=dev)
+            add(f"experts' first product, squared ReLU, tensor cores ({what})", "experts", lambda: K.expert_product_tc(ar, wu, h1, grp, cnt, act="relu2"),
+                used * I * D * 2 + N * top * (D + I) * 2, 2.0 * N * top * I * D)
+            add(f"experts' first product, gated SiLU, tensor cores, Pinorax ({what})", "", lambda: K.expert_product_tc(ar, wg, h2, grp, cnt, gated="silu"),
+                used * 2 * Ig * D * 2 + N * top * (D + Ig) * 2, 4.0 * N * top * Ig * D)
+        else:
+            h1, h2 = torch.empty(N * top, I, device=dev), torch.empty(N * top, Ig, device=dev)
+            add(f"experts' first product, squared ReLU, tiles of 16 rows ({what})", "experts", lambda: K.expert_product(xb, top, wu, h1, srt, grp, cnt, act="relu2"),
+                used * I * D * 2, simt=float(N * top * I * D))
+            add(f"experts' first product, gated SiLU, tiles of 16 rows, Pinorax ({what})", "",
+                lambda: K.expert_product(xb, top, wg, h2, srt, grp, cnt, gated="silu"), used * 2 * Ig * D * 2, simt=float(N * top * 2 * Ig * D))
+        Is = 3 * ff // 8
+        lu, lg = Linear(torch.randn(Is, D) * 0.02, bf, dev), Linear(torch.randn(2 * Is, D) * 0.02, bf, dev)
+        hs = torch.empty(N, Is, dtype=bf, device=dev)
+        add(f"shared expert's first product, squared ReLU ({what})", "gemm_swiglu", lambda: K.gemm_tc(xb, lu.weight, hs, w_tiles=lu.weight_tiles, act="relu2"),
+            Is * D * 2 + N * (D + Is) * 2, 2.0 * N * Is * D)
+        if n > 1:
+            add(f"shared expert's first product, gated SiLU, Pinorax ({what})", "", lambda: K.gemm_swiglu(xb, lg.weight, hs), 2 * Is * D * 2 + N * (D + Is) * 2,
+                4.0 * N * Is * D)
+        else:
+            gu = torch.empty(N, 2 * Is, device=dev)
+            add(f"shared expert's first product, gated SiLU in a second kernel, Pinorax ({what})", "",
+                lambda: (K.gemm_tc(xb, lg.weight, gu, w_tiles=lg.weight_tiles), K.swiglu(gu, hs)), 2 * Is * D * 2 + N * (D + Is) * 2)
+        # the product ahead of a pass: the half that is read per pass
+        lw = Linear(torch.randn(D, D) * 0.02, bf, dev)
+        add(f"W_x x added into the stream ({what})", "", lambda: lw.forward(xb, x, accumulate=True), D * D * 2 + N * D * 10, 2.0 * N * D * D)
+    return rows
+
+
+def run_mimolix(args):
+    """Prefill (one 2,048-token prompt in one step) and decode (batch 8 at context 2,048) throughput of Mimolix models whose
+    layers have the sizes of the Llama-3.2-1B and Llama-3.1-8B shapes (four layers each, random bf16 weights), beside Pinorax
+    (the closest existing design in its blocks and experts), Fovezen (the closest in its recurrence) and Llama models of the
+    same sizes; then every kernel that the design added or changed alone beside its like kernel. One JSON line."""
+    import torch
+    from geneinfer_b200 import Engine
+    from geneinfer_b200.weights import write_random_model
+    pk = peaks()
+    layers = args.layers or 4
+    context, batch, T = 2048, 8, PREFILL_TOKENS
+    models = []
+    for name, base in (("1b", LLAMA_1B), ("8b", LLAMA_8B)):
+        llama = dict(base, num_hidden_layers=layers, tie_word_embeddings=True)
+        width, ff, vocab, heads, hd = (base[k] for k in ("hidden_size", "intermediate_size", "vocab_size", "num_attention_heads", "head_dim"))
+        pin = pinorax_config(width, ff, layers, vocab, heads, hd, context)
+        fov = fovezen_config(width, ff, layers, vocab, heads, hd, base["num_key_value_heads"], 1024)
+        for arch, cfg in (("Llama", llama), ("Pinorax", pin), ("Fovezen", fov), ("Mimolix", mimolix_config(width, ff, layers, vocab, heads, hd))):
+            if arch == "Llama":
+                folder = model_folder(cfg)
+            else:
+                folder = os.path.join(tempfile.gettempdir(), f"geneinfer_bench_{arch.lower()}_{name}_{layers}_{context}_{os.getuid()}")
+                if not os.path.isfile(os.path.join(folder, "done")):
+                    write_random_model(cfg, 1, folder, "bfloat16", std=0.02)
+                    open(os.path.join(folder, "done"), "w").close()
+            llm = Engine(folder, dtype="bfloat16", max_seq_len=context, page_size=PAGE, kv_pages=batch * (context // PAGE),
+                         max_running=batch, step_tokens=T, prefix_cache=False)
+            ms_prefill = time_prefill(llm.steps, T, 2, vocab)
+            ms_decode, _ = time_decode_device(llm.steps, batch, context, args.steps, args.warmup, vocab)
+            llm.steps.check_status()
+            models.append({"model": f"{arch} at the {SHAPES[name][0]} layer sizes, {layers} layers",
+                           "prefill_2048_tok_s": round(T / ms_prefill * 1e3, 1), "prefill_ms": round(ms_prefill, 3),
+                           "decode_b8_ctx2048_tok_s": round(batch / ms_decode * 1e3, 1), "decode_ms_per_step": round(ms_decode, 4),
+                           "weight_gb": round(llm.model.weight_bytes() / 1e9, 3)})
+            del llm
+            torch.cuda.empty_cache()
+    table = mimolix_kernel_table(2048, 8192, 32, 64, T, pk)
+    print(json.dumps({"metric": "Mimolix beside Pinorax, Fovezen and Llama at equal layer sizes (random bf16 weights)", "impl": "ours", "n_gpus": 1,
+                      "dtype": "bf16", "steps": args.steps, "warmup": args.warmup, "peaks": pk["source"],
+                      "peak_gb_s": pk["hbm_gbs"], "peak_tflops": pk["bf16_tflops"], "models": models, "kernels": table}))
+    return 0
+
+
 def run_scenario(args):
     """Two workloads through the entry point, beside the default run: ``mixed`` (32 requests with
     prompts of 128 to 4096 random ids and 256 generated tokens each, admitted together, prompts cut
@@ -1432,7 +1646,7 @@ def main():
     ap.add_argument("--shape", choices=sorted(SHAPES), default="1b", help="layer sizes (the default is the baseline's third configuration)")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
                     help="precision of a --scenario run (float32: the requests run alone must give identical tokens)")
-    ap.add_argument("--scenario", choices=["mixed", "prefix", "sizes", "nipadra", "gekupel", "pinorax", "fovezen"], default="",
+    ap.add_argument("--scenario", choices=["mixed", "prefix", "sizes", "nipadra", "gekupel", "pinorax", "fovezen", "mimolix"], default="",
                     help="a workload through the scheduler (mixed, prefix) or decode steps at a grid of sizes, instead of the default run")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -1447,6 +1661,8 @@ def main():
         return run_nipadra(args)
     if args.scenario == "gekupel":
         return run_gekupel(args)
+    if args.scenario == "mimolix":
+        return run_mimolix(args)
     if args.scenario == "fovezen":
         return run_fovezen(args)
     if args.scenario == "pinorax":
