@@ -1287,9 +1287,10 @@ def mimolix_kernel_table(width, ff, heads, head_dim, T, pk):
         a_log, dt_bias = torch.zeros(H, device=dev), torch.full((H,), -3.0, device=dev)
         state = torch.zeros(R, H * dk * dv + 3 * C, device=dev)
         qkv, gates, out = torch.empty(N, C, device=dev), torch.empty(N, 2 * H, device=dev), torch.empty(N, H * dv, device=dev)
+        coefs = torch.empty(N, H, K.gated_delta_coefs(), device=dev) if K.gated_delta_in_blocks(N, R) else None
         step_bytes = N * (2 * C + C + H * dv) * 4 + 2 * R * (H * dk * dv + 3 * C) * 4
         add(f"gated_delta: convolution, unit norms, gates, recurrence ({what})", "linear_scan", lambda: K.gated_delta(
-            proj, 0, C + H * dv, C + H * dv + H, conv, a_log, dt_bias, 0.09, state, 0, H * dk * dv, rr, s0, sl, slots, qkv, gates, out, H, G, dk, dv),
+            proj, 0, C + H * dv, C + H * dv + H, conv, a_log, dt_bias, 0.09, state, 0, H * dk * dv, rr, s0, sl, slots, qkv, gates, out, H, G, dk, dv, coefs),
             step_bytes, simt=N * H * dk * dv * 4.0)
         cproj = torch.randn(N, C, device=dev)
         mixed = torch.empty(N, C, device=dev)

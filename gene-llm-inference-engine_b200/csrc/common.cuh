@@ -127,8 +127,10 @@ __device__ __forceinline__ float plain_value(float z, int act) {
     return z;
 }
 
+// ``early`` false: without that attribute. A kernel of about one long-running block per SM must not become resident while the
+// kernel ahead drains: its blocks would pile up on the SMs that happen to be free first and leave the others idle.
 template <typename... KArgs, typename... Args>
-inline void launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args&&... args) {
+inline void launch_kernel_as(bool early, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args&&... args) {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = block;
@@ -136,10 +138,14 @@ inline void launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_
     cfg.stream = stream;
     cudaLaunchAttribute attr[1];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = g_pdl_enabled ? 1 : 0;
+    attr[0].val.programmaticStreamSerializationAllowed = g_pdl_enabled && early ? 1 : 0;
     cfg.attrs = attr;
     cfg.numAttrs = 1;
     cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);      // errors surface in check_launch
+}
+template <typename... KArgs, typename... Args>
+inline void launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream, Args&&... args) {
+    launch_kernel_as(true, kernel, grid, block, smem, stream, std::forward<Args>(args)...);
 }
 
 // Launch programs. While a program is being recorded on the calling thread (gi_program_begin ..

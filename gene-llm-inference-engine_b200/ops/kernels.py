@@ -783,7 +783,7 @@ def gated_delta(proj: torch.Tensor, in_offset: int, b_offset: int, a_offset: int
                 dt_bias: torch.Tensor, q_scale: float, state: torch.Tensor, state_offset: int, conv_offset: int,
                 row_req: torch.Tensor, seg_start: torch.Tensor, seg_len: torch.Tensor, state_slots: torch.Tensor, qkv: torch.Tensor,
                 gates: torch.Tensor, out: torch.Tensor, num_heads: int, key_heads: int, dk: int, dv: int,
-                narrow: Optional[bool] = None, unit_eps: float = 1e-6) -> None:
+                coefs: Optional[torch.Tensor] = None, unit_eps: float = 1e-6) -> None:
     """The gated delta rule over each request's rows in order. ``proj`` [T, ld] holds the projections of q, k (key_heads of
     dk) and v (H heads of dv) side by side from in_offset and those of b and a (H each). q, k and v pass a causal convolution
     (``conv`` [channels, taps], the last column weighs the token itself; its last taps - 1 inputs are the block [taps - 1,
@@ -791,8 +791,8 @@ def gated_delta(proj: torch.Tensor, in_offset: int, b_offset: int, a_offset: int
     unit_eps), q multiplied by q_scale; beta = sigmoid(b), g = exp(-exp(a_log) softplus(a + dt_bias)). Then per head (which
     reads key head h // (H / key_heads)), with the state S [dk, dv] at state_offset of the slot: S <- g S;
     u = beta (v - S^T k); S <- S + k u^T; ``out``[t, h] = S^T q. ``qkv`` [T, channels] and ``gates`` [T, 2 H] are workspaces.
-    ``narrow``: how a head's columns are spread (see the kernel; chosen by the rows per request when None); results are the
-    same bit for bit. Two launches."""
+    ``coefs`` [T, H, gated_delta_coefs()], a further workspace: the recurrence runs in blocks of eight tokens (faster for long
+    portions); without it token by token. The two differ by rounding only. Two launches, in blocks three."""
     T, ld = proj.shape
     C, taps = conv.shape
     if C != 2 * key_heads * dk + num_heads * dv or qkv.shape != (T, C) or gates.shape != (T, 2 * num_heads) or out.shape != (T, num_heads * dv):
@@ -803,16 +803,26 @@ def gated_delta(proj: torch.Tensor, in_offset: int, b_offset: int, a_offset: int
             conv_offset + (taps - 1) * C > state.shape[1]:
         raise KernelError("gated_delta: the state does not fit the slot")
     R = seg_start.numel()
-    if narrow is None:
-        narrow = T > 4 * R
+    if coefs is not None and coefs.shape != (T, num_heads, gated_delta_coefs()):
+        raise KernelError("gated_delta: coefs must be [T, H, gated_delta_coefs()]")
     check(lib().gi_gated_delta(
         _dev(proj, "proj", torch.float32), ld, int(in_offset), int(b_offset), int(a_offset), _dev(conv, "conv", torch.float32), taps,
         _dev(a_log, "a_log", torch.float32), _dev(dt_bias, "dt_bias", torch.float32), float(q_scale), float(unit_eps),
         _dev(state, "state", torch.float32), state.shape[1], int(state_offset), int(conv_offset), _dev(row_req, "row_req", torch.int32),
         _dev(seg_start, "seg_start", torch.int32), _dev(seg_len, "seg_len", torch.int32), _dev(state_slots, "state_slots", torch.int32),
-        _dev(qkv, "qkv", torch.float32), _dev(gates, "gates", torch.float32), _dev(out, "out", torch.float32), T, R, num_heads,
-        key_heads, dk, dv, int(bool(narrow)), _stream()), "gated_delta")
-    count_launches(1)
+        _dev(qkv, "qkv", torch.float32), _dev(gates, "gates", torch.float32), _opt(coefs, "coefs", torch.float32),
+        _dev(out, "out", torch.float32), T, R, num_heads, key_heads, dk, dv, _stream()), "gated_delta")
+    count_launches(1 if coefs is None else 2)
+
+
+def gated_delta_coefs() -> int:
+    """Coefficients per token and head that the recurrence in blocks keeps in its workspace."""
+    return int(lib().gi_gated_delta_coefs())
+
+
+def gated_delta_in_blocks(T: int, R: int) -> bool:
+    """Whether a step of T tokens of R requests is better off with the recurrence in blocks of tokens."""
+    return T > 4 * R
 
 
 def linear_scan(q: torch.Tensor, q_offset: int, k: torch.Tensor, k_offset: int, v: torch.Tensor, v_offset: int,

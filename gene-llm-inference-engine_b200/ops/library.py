@@ -69,8 +69,9 @@ _SIGNATURES = {
                            c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "gi_maps_combine": [c_void_p, c_int, c_void_p, c_int, c_float, c_float, c_float, c_int, c_int, c_int, c_void_p],
     "gi_gated_delta": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p,
-                       c_longlong, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                       c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+                       c_longlong, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                       c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "gi_gated_delta_coefs": [],
     "gi_streams": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p,
                    c_int, c_int, c_int, c_void_p],
     "gi_grouped_tile_rows": [],

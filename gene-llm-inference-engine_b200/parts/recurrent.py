@@ -331,10 +331,13 @@ class GatedDeltaMixer:
         qkv = ctx.scratch("delta_qkv", (T, C), torch.float32)
         gates = ctx.scratch("delta_gates", (T, 2 * H), torch.float32)
         o = ctx.scratch("delta_out", (T, H * dv), torch.float32)
+        coefs = None
+        if kernels.gated_delta_in_blocks(T, ctx.n_requests):
+            coefs = ctx.scratch("delta_coefs", (T, H, kernels.gated_delta_coefs()), torch.float32)
         b = C + H * dv
         kernels.gated_delta(proj, 0, b, b + H, self.conv, self.a_log, self.dt_bias, self.q_scale, ctx.state(run.cache_layer),
                             self.state_offset, self.state_offset + H * dk * dv, ctx.row_req, ctx.seg_start, ctx.seg_len,
-                            ctx.state_slots, qkv, gates, o, H, self.key_heads, dk, dv)
+                            ctx.state_slots, qkv, gates, o, H, self.key_heads, dk, dv, coefs)
         y = ctx.scratch("delta_normed", (T, H * dv), self.dtype)
         kernels.gated_group_norm(o, proj, C, self.norm, y, H, self.eps, gate_first=False, gate_act="silu", out_scale=self.out_scale)
         self.w_o.forward(y, x, accumulate=True, then=then)

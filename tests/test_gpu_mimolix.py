@@ -227,7 +227,7 @@ def _plain_delta(rows, conv, a_log, dt_bias, H, G, dk, dv, q_scale):
     return px.delta_rule(q, k, x[:, 2 * G * dk:].reshape(T, H, dv), beta, decay)
 
 
-def _run_delta(seqs, cuts, conv, a_log, dt_bias, H, G, dk, dv, q_scale, slots, narrow=None, lead=5):
+def _run_delta(seqs, cuts, conv, a_log, dt_bias, H, G, dk, dv, q_scale, slots, blocks=None, lead=5):
     """Feeds the rows of ``seqs`` through the kernel under ``cuts``; returns outputs and the whole state tensor."""
     from geneinfer_b200.ops import kernels
     C, taps = conv.shape
@@ -244,9 +244,11 @@ def _run_delta(seqs, cuts, conv, a_log, dt_bias, H, G, dk, dv, q_scale, slots, n
         i32 = lambda v: torch.tensor([int(x) for x in v], dtype=torch.int32, device=DEV)
         out = torch.full((T, H * dv), float("nan"), device=DEV)
         qkv, gates = torch.full((T, C), float("nan"), device=DEV), torch.full((T, 2 * H), float("nan"), device=DEV)
+        in_blocks = kernels.gated_delta_in_blocks(T, len(live)) if blocks is None else blocks
+        coefs = torch.full((T, H, kernels.gated_delta_coefs()), float("nan"), device=DEV) if in_blocks else None
         kernels.gated_delta(rows, 0, C, C + H, conv.to(DEV), a_log.to(DEV), dt_bias.to(DEV), q_scale, state, lead, floats, row_req,
                             i32(starts[:-1]), i32([lengths[r] for r in live]), i32([slots[r] for r in live]), qkv, gates, out, H, G, dk, dv,
-                            narrow=narrow)
+                            coefs)
         for i, r in enumerate(live):
             got[r].append(out[starts[i]:starts[i + 1]].cpu())
             at[r] += lengths[r]
@@ -256,8 +258,8 @@ def _run_delta(seqs, cuts, conv, a_log, dt_bias, H, G, dk, dv, q_scale, slots, n
 @pytest.mark.parametrize("H, G, dk, dv, taps", [(4, 2, 16, 24, 3), (3, 3, 40, 33, 1), (6, 1, 64, 64, 4), (2, 2, 100, 20, 5), (2, 1, 128, 96, 2),
                                                 (1, 1, 200, 72, 4), (2, 2, 7, 5, 17), (8, 4, 96, 128, 4)])
 def test_gated_delta_kernel(H, G, dk, dv, taps):
-    """Outputs, the state and the convolution's inputs left in the slots, against the plain recurrence; and the same bits
-    whichever way the requests are cut and a head's columns are spread."""
+    """Outputs, the state and the convolution's inputs left in the slots, against the plain recurrence, token by token and in
+    blocks of eight (whose last one may not be whole); token by token the same bits whichever way the requests are cut."""
     g = torch.Generator().manual_seed(H * 100 + dk)
     conv = torch.randn(2 * G * dk + H * dv, taps, generator=g) * 0.6
     a_log, dt_bias = torch.rand(H, generator=g) * 2 - 1, torch.randn(H, generator=g) - 2
@@ -267,9 +269,10 @@ def test_gated_delta_kernel(H, G, dk, dv, taps):
     want = [_plain_delta(s, *args) for s in seqs]
     slots = [3, 0, 1]
     base = None
-    for cuts, narrow in (([[90, 2, 37]], True), ([[90, 2, 37]], False), ([[1, 1, 1], [40, 1, 2], [2, 0, 1], [47, 0, 33]], None),
+    ragged = [[1, 1, 1], [40, 1, 2], [2, 0, 1], [47, 0, 33]]
+    for cuts, blocks in (([[90, 2, 37]], True), ([[90, 2, 37]], False), (ragged, True), (ragged, False), (ragged, None),
                          ([[2, 0, 0], [0, 2, 3]] + [[1, 0, 1]] * 34 + [[54, 0, 0]], None)):
-        got, state = _run_delta(seqs, cuts, *args, slots, narrow)
+        got, state = _run_delta(seqs, cuts, *args, slots, blocks)
         for r in range(3):
             _close(got[r], want[r][0].reshape(lens[r], H * dv), torch.float32, f"outputs of request {r}, {len(cuts)} steps", f32=1e-5)
             _close(state[slots[r], 5:5 + H * dk * dv], want[r][1].reshape(-1), torch.float32, f"state of request {r}", f32=1e-5)
@@ -279,9 +282,9 @@ def test_gated_delta_kernel(H, G, dk, dv, taps):
                 kept[taps - 1 - tail.shape[0]:] = tail
                 assert torch.equal(state[slots[r], -(taps - 1) * conv.shape[0]:].view(taps - 1, -1), kept)
         assert not state[:, :5].any() and not state[2].any() and not state[4].any()
-        if base is None:
-            base = got, state
-        assert all(torch.equal(a, b) for a, b in zip(got, base[0])) and torch.equal(state, base[1])
+        if blocks is False:
+            base = base or (got, state)
+            assert all(torch.equal(a, b) for a, b in zip(got, base[0])) and torch.equal(state, base[1])
 
 
 def test_gated_delta_remembers_replaces_and_forgets():
@@ -487,7 +490,8 @@ def test_the_first_tokens_see_zeros_before_the_sequence_through_the_convolution(
 
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_requests_in_one_batch_equal_each_alone(dtype):
-    """Three unequal requests batched against each alone, on scattered pages and other state slots: the same bits."""
+    """Three unequal requests batched against each alone, on scattered pages and other state slots: the same bits (the
+    recurrence may run in blocks of tokens in one and token by token in the other: equal but for rounding)."""
     D = 40
     g = torch.Generator().manual_seed(17)
     fast = dict(MAPS, dim=32, vdim=64)
@@ -499,7 +503,10 @@ def test_requests_in_one_batch_equal_each_alone(dtype):
         together = _run_mixer(part, ctx_of(3), inputs, [[20, 1, 3], [1, 1, 2], [12, 3, 7]], dtype, D)
         for r in range(3):
             alone = _run_mixer(part, ctx_of(1), [inputs[r]], [[[20, 1, 3][r]], [[1, 1, 2][r]], [[12, 3, 7][r]]], dtype, D)
-            assert torch.equal(alone[0], together[r]), f"request {r} depends on its batch"
+            if part is delta_part:
+                _close(alone[0], together[r], dtype, f"request {r} in a batch", f32=1e-5, b16=1e-2)
+            else:
+                assert torch.equal(alone[0], together[r]), f"request {r} depends on its batch"
 
 
 # ------------------------------------------------------------------------------------------ whole models
