@@ -1346,6 +1346,26 @@ def mimolix_kernel_table(width, ff, heads, head_dim, T, pk):
             R * seen * AH * 2.0 * (2 * dim + 2 * vd))
         add(f"attention, plain heads, Fovezen ({what})", "", lambda: attend(both, 2 * AH), cache_bytes + N * 2 * AH * vd * 4,
             R * seen * 2 * AH * 4.0 * head_dim)
+        both32 = torch.empty(N, 2 * AH * vd, device=dev)
+
+        class Ctx:                      # what attention_rows_of_step reads of a step
+            row_req, positions, page_size, max_position, kept = rr, pos, page, T, {}
+
+            @staticmethod
+            def scratch(name, shape, dtype, capacity=None):
+                key = (name, tuple(shape), dtype)
+                if key not in Ctx.kept:
+                    Ctx.kept[key] = torch.empty(shape, dtype=dtype, device=dev)
+                return Ctx.kept[key]
+
+            @staticmethod
+            def attention_work(per_tile):
+                if n == 1:
+                    return rows_dec, work[:0], T
+                return rows_dec[:0], torch.tensor([(t, min(per_tile, n - t), 0) for t in range(0, n, per_tile)], **i32), 0
+        add(f"attention, two maps, row-form kernel, where other sizes run ({what})", "attention", lambda: K.attention_rows_of_step(
+            Ctx, q, kc, vc, both32, tables, 2 * AH, AG, head_dim, vd, 0.1, None, None, None, None), cache_bytes + N * 2 * AH * vd * 6,
+            R * seen * AH * 2.0 * (2 * dim + 2 * vd))
         add(f"maps_combine ({what})", "gated_group_norm", lambda: K.maps_combine(both, att, 0.5, 1e-6, 0.5, AH), N * AH * vd * 6)
         # routing and experts
         E, top = 8, 2

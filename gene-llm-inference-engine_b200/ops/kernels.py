@@ -275,15 +275,18 @@ def maps_norm_store(proj: torch.Tensor, q_offset: int, k_offset: int, v_offset: 
     """Heads of two score maps: from the 32-bit projections ``proj`` [T, ld] (from q_offset H heads of [map 1, map 2], dim
     values each; from k_offset G such heads; from v_offset G value heads), every map is brought to unit RMS and weighted by
     ``q_norm`` / ``k_norm`` [dim]; with ``temperature`` (coef, every) the queries at position p are multiplied by
-    1 + coef ln(floor((p + 1) / every) + 1). ``q_out`` [T, H * 2 * 2 dim]: row [map 1, 0], then row [0, map 2] per head; keys
-    into the token's row of ``k_cache`` [pages, G, page_size, 2 dim], values into ``v_cache`` [pages, G, page_size, value_dim]."""
+    1 + coef ln(floor((p + 1) / every) + 1). ``q_out`` [T, H * 2 * w]: row [map 1, 0], then row [0, map 2] per head; keys
+    into the token's row of ``k_cache`` [pages, G, page_size, w], values into ``v_cache`` [pages, G, page_size, wv]; w >= 2 dim
+    and wv >= value_dim, with zeros behind."""
     T, ld = proj.shape
-    if q_out.shape != (T, num_heads * 4 * dim):
-        raise KernelError("maps_norm_store: q_out must be [T, H * 2 * 2 dim]")
+    w, wv = k_cache.shape[-1], v_cache.shape[-1]
+    if q_out.shape != (T, num_heads * 2 * w):
+        raise KernelError("maps_norm_store: q_out must be [T, H * 2 * w]")
     if k_cache.dtype != q_out.dtype or v_cache.dtype != q_out.dtype:
         raise KernelError("maps_norm_store: q_out and the cache must have one dtype")
-    if k_cache.shape[1:] != (num_kv_heads, page_size, 2 * dim) or v_cache.shape != (k_cache.shape[0], num_kv_heads, page_size, value_dim):
-        raise KernelError("maps_norm_store: the cache must be [pages, G, page_size, 2 dim] (values: their own width)")
+    if k_cache.shape[1:] != (num_kv_heads, page_size, w) or v_cache.shape != (k_cache.shape[0], num_kv_heads, page_size, wv) or \
+            w < 2 * dim or wv < value_dim:
+        raise KernelError("maps_norm_store: the cache must be [pages, G, page_size, at least 2 dim] (values: their own width)")
     if q_norm.numel() != dim or k_norm.numel() != dim:
         raise KernelError("maps_norm_store: the norms' weights must have dim values")
     coef, every = temperature if temperature is not None else (0.0, 1.0)
@@ -292,7 +295,7 @@ def maps_norm_store(proj: torch.Tensor, q_offset: int, k_offset: int, v_offset: 
         _dev(k_norm, "k_norm", torch.float32), float(eps), float(coef), float(every), _dev(positions, "positions", torch.int32),
         _dev(row_req, "row_req", torch.int32), _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1],
         _dev(q_out, "q_out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), dtype_code(q_out.dtype), T, num_heads, num_kv_heads,
-        dim, value_dim, page_size, int(write_kv), _stream()), "maps_norm_store")
+        dim, value_dim, w, wv, page_size, int(write_kv), _stream()), "maps_norm_store")
 
 
 def maps_combine_supported(value_dim: int) -> bool:
@@ -300,14 +303,14 @@ def maps_combine_supported(value_dim: int) -> bool:
 
 
 def maps_combine(a: torch.Tensor, out: torch.Tensor, weight: float, eps: float, factor: float, num_heads: int) -> None:
-    """``a`` [T, H * 2 * vd] holds two outputs a1, a2 per head: out[t, h] = factor * N(a1 - weight * a2), N to unit RMS over the
-    vd values."""
+    """``a`` [T, H * 2 * wv] holds two outputs a1, a2 per head, the first vd values of rows of wv: out[t, h] = factor * N(a1 -
+    weight * a2), N to unit RMS over the vd values; ``out`` [T, H * vd]."""
     T = a.shape[0]
-    vd = out.shape[1] // num_heads
-    if out.shape != (T, num_heads * vd) or a.shape != (T, 2 * num_heads * vd):
-        raise KernelError("maps_combine: a must be [T, H * 2 * vd] for out [T, H * vd]")
+    vd, wv = out.shape[1] // num_heads, a.shape[1] // (2 * num_heads)
+    if out.shape != (T, num_heads * vd) or a.shape != (T, 2 * num_heads * wv) or wv < vd:
+        raise KernelError("maps_combine: a must be [T, H * 2 * wv] for out [T, H * vd]")
     check(lib().gi_maps_combine(_dev(a, "a"), dtype_code(a.dtype), _dev(out, "out"), dtype_code(out.dtype), float(weight), float(eps),
-                                float(factor), T, num_heads, vd, _stream()), "maps_combine")
+                                float(factor), T, num_heads, vd, wv, _stream()), "maps_combine")
 
 
 def add_normed(y: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, eps: float, xn_out: Optional[torch.Tensor] = None,

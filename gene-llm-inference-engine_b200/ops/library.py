@@ -66,8 +66,8 @@ _SIGNATURES = {
     "gi_plain_act": [c_void_p, c_void_p, c_int, c_longlong, c_int, c_void_p],
     "gi_take_stream": [c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_void_p],
     "gi_maps_norm_store": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_float, c_void_p, c_void_p,
-                           c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "gi_maps_combine": [c_void_p, c_int, c_void_p, c_int, c_float, c_float, c_float, c_int, c_int, c_int, c_void_p],
+                           c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "gi_maps_combine": [c_void_p, c_int, c_void_p, c_int, c_float, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p],
     "gi_gated_delta": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p,
                        c_longlong, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                        c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],

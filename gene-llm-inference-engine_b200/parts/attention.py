@@ -51,7 +51,9 @@ class AttentionMixer:
     map_weight (weights ``lq1``, ``lk1``, ``lq2``, ``lk2`` [hd]), a head's output is map_factor * N(a1 - w a2), N to unit RMS over the
     value width (eps ``qk_norm_eps``). ``query_temperature`` (coef, every): the queries at position p are multiplied by
     1 + coef ln(floor((p + 1) / every) + 1). The cache holds [map 1, map 2] in one key row per key head; to the attention
-    kernels these are 2 H query heads ([map 1, 0] and [0, map 2]) over Hkv key heads of 2 hd, which share the rows they read."""
+    kernels these are 2 H query heads ([map 1, 0] and [0, map 2]) over Hkv key heads of 2 hd, which share the rows they read.
+    In bfloat16, rows of keys and values are widened with zeros to a width that the tensor-core kernels are built for where that
+    at most doubles them; other sizes and the 32-bit path run the row-form kernel."""
 
     graph_safe = True      # launches depend only on the step's shape: decode steps may be captured in a CUDA graph
 
@@ -80,7 +82,8 @@ class AttentionMixer:
         if params.get("values", "projected") not in ("projected", "keys"):
             raise ValueError(f"attention: unknown source of values '{params.get('values')}'")
         self.qk_norm_eps = params.get("qk_norm_eps")
-        self.value_dim = int(params.get("value_dim") or params["head_dim"])
+        if self.maps == 1:
+            self.value_dim = int(params.get("value_dim") or self.head_dim)
         self.chunk = params.get("chunk")
         self.learned_sink = params.get("sink") == "learned"
         self.softcap = float(params["softcap"]) if params.get("softcap") else None
@@ -140,13 +143,17 @@ class AttentionMixer:
                 setattr(self, name, weights[name].to(device=build.device, dtype=torch.float32).contiguous())
         if self.wide_norm and (self.qk_norm_eps is None or not params.get("qk_norm_weights", True)):
             raise ValueError("attention: qk_norm_wide needs qk_norm_eps and weights")
-        query_rows = self.num_heads * self.head_dim // self.maps
-        qkv_rows = query_rows + self.num_kv_heads * self.head_dim + \
-            (0 if self.values_are_keys else self.num_kv_heads * self.value_dim) + (self.num_heads if self.head_gate else 0)
+        if self.maps == 2:
+            qkv_rows = 2 * (self.map_heads + self.num_kv_heads) * self.map_dim + self.num_kv_heads * self.map_value_dim
+            out_columns = self.map_heads * self.map_value_dim
+        else:
+            qkv_rows = (self.num_heads + self.num_kv_heads) * self.head_dim + \
+                (0 if self.values_are_keys else self.num_kv_heads * self.value_dim) + (self.num_heads if self.head_gate else 0)
+            out_columns = self.num_heads * self.value_dim
         if tuple(weights["w_qkv"].shape) != (qkv_rows, self.hidden_size):
             raise ValueError(f"attention: w_qkv has shape {tuple(weights['w_qkv'].shape)}, expected "
                              f"({qkv_rows}, {self.hidden_size})")
-        if tuple(weights["w_o"].shape) != (self.hidden_size, self.num_heads // self.maps * self.value_dim):
+        if tuple(weights["w_o"].shape) != (self.hidden_size, out_columns):
             raise ValueError(f"attention: w_o has shape {tuple(weights['w_o'].shape)}")
         self.conv = None
         if self.conv_taps is not None:
@@ -181,8 +188,14 @@ class AttentionMixer:
         if params.get("qk_norm_eps") is None or not params.get("qk_norm_weights", True):
             raise ValueError("attention: two score maps need qk_norm_eps and weights")
         self.map_heads, self.map_dim = self.num_heads, self.head_dim
-        self.num_heads, self.head_dim = 2 * self.num_heads, 2 * self.head_dim
-        vd = int(params.get("value_dim") or self.map_dim)
+        vd = self.map_value_dim = int(params.get("value_dim") or self.map_dim)
+        self.num_heads, self.head_dim, self.value_dim = 2 * self.num_heads, 2 * self.head_dim, vd
+        if build.compute_dtype is torch.bfloat16:
+            widest = max(self.head_dim, vd)
+            width = next((w for w in (16, 32, 64, 128) if w >= widest), None)
+            if width and 2 * width <= 2 * (self.head_dim + vd) and \
+                    kernels.attention_fast_supported(width, self.num_heads, self.num_kv_heads):
+                self.head_dim = self.value_dim = width
         if not kernels.attention_rows_supported(self.head_dim, vd) or not kernels.maps_combine_supported(vd):
             raise ValueError(f"attention: two maps of size {self.map_dim} with value size {vd} are not supported")
         lq1, lk1, lq2, lk2 = (_vector_of(weights, n, self.map_dim, build).double() for n in ("lq1", "lk1", "lq2", "lk2"))
@@ -320,15 +333,16 @@ class AttentionMixer:
             kernels.causal_conv(proj, 0, self.conv, None, state, self.state_offset if self.conv_taps > 1 else 0, ctx.row_req,
                                 ctx.seg_start, ctx.seg_len, ctx.state_slots, mixed, activate=False)
             proj = mixed
-        k_off = H * hd // self.maps
-        v_off = k_off if self.values_are_keys else k_off + Hkv * hd
-        gate_off = v_off + Hkv * hd
         if self.maps == 2:
-            kernels.maps_norm_store(proj, 0, k_off, v_off, self.q_norm, self.k_norm, self.qk_norm_eps, self.temperature, ctx.positions,
-                                    ctx.row_req, tables, q, k_cache, v_cache, self.map_heads, Hkv, self.map_dim, self.value_dim,
-                                    ctx.page_size, write_kv=run.writes_cache)
+            k_off = 2 * self.map_heads * self.map_dim
+            kernels.maps_norm_store(proj, 0, k_off, k_off + 2 * Hkv * self.map_dim, self.q_norm, self.k_norm, self.qk_norm_eps,
+                                    self.temperature, ctx.positions, ctx.row_req, tables, q, k_cache, v_cache, self.map_heads, Hkv,
+                                    self.map_dim, self.map_value_dim, ctx.page_size, write_kv=run.writes_cache)
             self._attend_maps(ctx, q, k_cache, v_cache, tables, x, then)
             return
+        k_off = H * hd
+        v_off = k_off if self.values_are_keys else k_off + Hkv * hd
+        gate_off = v_off + Hkv * hd
         kernels.norm_rope_store(proj, 0, k_off, v_off, self.q_norm, self.k_norm, self.qk_norm_eps or 0.0,
                                 getattr(self.position, "freq", None), self.position.interleaved, ctx.positions,
                                 ctx.row_req, tables, q, k_cache, v_cache, H, Hkv, hd, ctx.page_size,
@@ -369,7 +383,7 @@ class AttentionMixer:
         else:
             both = ctx.scratch("att_maps", (T, H * vd), self.dtype)
             self._attend(ctx, q, k_cache, v_cache, both, tables)
-        att = ctx.scratch("att", (T, self.map_heads * vd), self.dtype)
+        att = ctx.scratch("att", (T, self.map_heads * self.map_value_dim), self.dtype)
         kernels.maps_combine(both, att, self.map_weight, self.qk_norm_eps, self.map_factor, self.map_heads)
         self.w_o.forward(att, x, accumulate=True, then=then)
 

@@ -95,8 +95,10 @@ def test_end_of_a_layer_with_a_layer_norm_or_a_hand_over(dtype, D):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("more", [0, 5])
 @pytest.mark.parametrize("H, G, dim, vd, temp", [(4, 2, 16, 24, (0.5, 3)), (2, 2, 7, 10, None), (6, 1, 40, 96, (0.3, 1)), (2, 1, 128, 64, (-0.1, 2.5))])
-def test_maps_norm_and_store(dtype, H, G, dim, vd, temp):
+def test_maps_norm_and_store(dtype, H, G, dim, vd, temp, more):
+    """``more``: how much wider the rows of queries and keys (values: twice that) are than what they hold."""
     from geneinfer_b200.ops import kernels
     g = torch.Generator().manual_seed(H * 7 + dim)
     T, page = 11, 4
@@ -104,8 +106,9 @@ def test_maps_norm_and_store(dtype, H, G, dim, vd, temp):
     proj = torch.randn(T, ld, generator=g) * 2
     qw, kw = torch.randn(dim, generator=g), torch.randn(dim, generator=g)
     tables = torch.tensor([[2, 0, 1]], dtype=torch.int32)
-    q = torch.full((T, 4 * H * dim), float("nan"), dtype=dtype, device=DEV)
-    kc, vc = (torch.full((3, G, page, n), float("nan"), dtype=dtype, device=DEV) for n in (2 * dim, vd))
+    w, wv = 2 * dim + more, vd + 2 * more
+    q = torch.full((T, 2 * H * w), float("nan"), dtype=dtype, device=DEV)
+    kc, vc = (torch.full((3, G, page, n), float("nan"), dtype=dtype, device=DEV) for n in (w, wv))
     kernels.maps_norm_store(proj.to(DEV), 3, 3 + 2 * H * dim, 3 + 2 * (H + G) * dim, qw.to(DEV), kw.to(DEV), EPS, temp,
                             torch.arange(T, dtype=torch.int32, device=DEV), torch.zeros(T, dtype=torch.int32, device=DEV), tables.to(DEV), q,
                             kc, vc, H, G, dim, vd, page)
@@ -113,14 +116,15 @@ def test_maps_norm_and_store(dtype, H, G, dim, vd, temp):
     pk = px.unit_rms(proj[:, 3 + 2 * H * dim:3 + 2 * (H + G) * dim].double().view(T, G, 2, dim), EPS) * kw
     if temp:
         pq = pq * px.query_temperature(T, *temp, F)[:, None, None, None]
-    rows = torch.zeros(T, H, 2, 2, dim, dtype=F)
-    rows[:, :, 0, 0], rows[:, :, 1, 1] = pq[:, :, 0], pq[:, :, 1]
-    _close(q.cpu().float().view(T, H, 2, 2, dim), rows, dtype, "query rows", f32=5e-6, b16=1e-2)
+    rows = torch.zeros(T, H, 2, w, dtype=F)
+    rows[:, :, 0, :dim], rows[:, :, 1, dim:2 * dim] = pq[:, :, 0], pq[:, :, 1]
+    _close(q.cpu().float().view(T, H, 2, w), rows, dtype, "query rows", f32=5e-6, b16=1e-2)
     order = [2, 0, 1]
     keys = torch.stack([kc[order[t // page], :, t % page].cpu().float() for t in range(T)])
     vals = torch.stack([vc[order[t // page], :, t % page].cpu().float() for t in range(T)])
-    _close(keys, pk.reshape(T, G, 2 * dim), dtype, "keys in their pages", f32=5e-6, b16=1e-2)
-    _close(vals, proj[:, 3 + 2 * (H + G) * dim:].view(T, G, vd), dtype, "values in their pages", f32=1e-7, b16=1e-2)
+    pad = torch.nn.functional.pad
+    _close(keys, pad(pk.reshape(T, G, 2 * dim), (0, more)), dtype, "keys in their pages", f32=5e-6, b16=1e-2)
+    _close(vals, pad(proj[:, 3 + 2 * (H + G) * dim:].view(T, G, vd), (0, 2 * more)), dtype, "values in their pages", f32=1e-7, b16=1e-2)
 
 
 @pytest.mark.parametrize("out_dtype", DTYPES)
@@ -129,10 +133,10 @@ def test_maps_norm_and_store(dtype, H, G, dim, vd, temp):
 def test_maps_combine(in_dtype, out_dtype, H, vd):
     from geneinfer_b200.ops import kernels
     g = torch.Generator().manual_seed(vd)
-    a = torch.randn(6, H, 2, vd, generator=g).to(in_dtype)
+    a = torch.randn(6, H, 2, vd + 3, generator=g).to(in_dtype)           # rows wider than what they hold
     out = torch.full((6, H * vd), float("nan"), dtype=out_dtype, device=DEV)
     kernels.maps_combine(a.view(6, -1).to(DEV), out, 0.83, 1e-3, 0.4, H)
-    want = px.difference_of_maps(a[:, :, 0].double(), a[:, :, 1].double(), 0.83, 0.6, 1e-3)
+    want = px.difference_of_maps(a[:, :, 0, :vd].double(), a[:, :, 1, :vd].double(), 0.83, 0.6, 1e-3)
     _close(out.cpu().float(), want.reshape(6, -1), out_dtype, "difference of the maps", f32=3e-6, b16=1e-2)
 
 
@@ -332,7 +336,10 @@ MAPS_FORMS = [MAPS, dict(MAPS, heads=3, kv_heads=3, dim=10, vdim=14, q_temp=None
               dict(MAPS, heads=4, kv_heads=2, dim=16, vdim=32), dict(MAPS, heads=4, kv_heads=2, dim=32, vdim=64, diff=0.7),
               dict(MAPS, heads=2, kv_heads=1, dim=64, vdim=128, scale=0.2), dict(MAPS, heads=16, kv_heads=1, dim=32, vdim=64),
               # the row-form kernel's sizes: values in whole 64s, rows of two maps in whole 16s
-              dict(MAPS, heads=8, kv_heads=2, dim=40, vdim=64), dict(MAPS, heads=8, kv_heads=1, dim=64, vdim=192),
+              dict(MAPS, heads=20, kv_heads=2, dim=40, vdim=64), dict(MAPS, heads=8, kv_heads=1, dim=64, vdim=192),
+              # widened with zeros in bfloat16: keys to the values' width, values to the keys', both; too narrow to be widened
+              dict(MAPS, heads=4, kv_heads=2, dim=20, vdim=64), dict(MAPS, heads=4, kv_heads=4, dim=64, vdim=40),
+              dict(MAPS, heads=6, kv_heads=3, dim=36, vdim=80), dict(MAPS, heads=3, kv_heads=1, dim=34, vdim=20),
               dict(MAPS, heads=2, kv_heads=2, dim=136, vdim=200)]
 
 
@@ -356,8 +363,9 @@ def _maps_part(D, m, w, dtype, p="p.", eps=EPS):
                                 "query_temperature": (temp["coef"], temp["every"]) if temp else None}, weights, _build(dtype))
 
 
-def _maps_ctx(m, dtype, n, max_len=256, page_size=8):
-    return StateCtx(dtype, n, Hkv=m["kv_heads"], hd=2 * m["dim"], vd=m["vdim"], page_size=page_size, max_len=max_len)
+def _maps_ctx(part, dtype, n, max_len=256, page_size=8):
+    need = part.cache_need()
+    return StateCtx(dtype, n, Hkv=need.num_kv_heads, hd=need.head_dim, vd=need.value_width, page_size=page_size, max_len=max_len)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -369,13 +377,14 @@ def test_attention_with_two_score_maps(dtype, m, cut):
     w = _maps_weights(D, m, g)
     part = _maps_part(D, m, w, dtype)
     need = part.cache_need()
-    assert (need.num_kv_heads, need.head_dim, need.value_width) == (m["kv_heads"], 2 * m["dim"], m["vdim"])
-    fast = dtype is torch.bfloat16 and 2 * m["dim"] == m["vdim"] and m["vdim"] in (32, 64, 128) and 2 * m["heads"] // m["kv_heads"] <= 16
+    width = next((w for w in (16, 32, 64, 128) if w >= max(2 * m["dim"], m["vdim"])), 0)
+    fast = dtype is torch.bfloat16 and width > 0 and width <= 2 * m["dim"] + m["vdim"] and 2 * m["heads"] // m["kv_heads"] <= 16
     assert part.fast == fast and part.row_form != fast
+    assert (need.num_kv_heads, need.head_dim, need.value_width) == (m["kv_heads"], *((width, width) if fast else (2 * m["dim"], m["vdim"])))
     inputs = [_bf(torch.randn(n, D, generator=g)) for n in (40, 2, 19)]
     rnd = px.ident if dtype is torch.float32 else px.bf16
     want = [px.attention_mixer(w, "p.", m, x.double(), EPS, F, rnd) for x in inputs]
-    got = _run_mixer(part, _maps_ctx(m, dtype, 3), inputs, CUTS[cut], dtype, D)
+    got = _run_mixer(part, _maps_ctx(part, dtype, 3), inputs, CUTS[cut], dtype, D)
     for r in range(3):
         _close(got[r], want[r], dtype, f"two maps, request {r}, {cut}", b16=3e-2)
 
@@ -416,7 +425,7 @@ def test_one_key_among_hundreds_in_one_map(dtype, which, back, form):
     assert float((px.attention_mixer(w, "p.", m, moved.double(), EPS, F, rnd)[-1] - want[-1]).abs().max()) > 0.1 * float(want[-1].abs().max())
     part = _maps_part(D, m, w, dtype)
     for cuts in ([[n - 30]] + [[1]] * 30, [[300], [398], [2]]):
-        got = _run_mixer(part, _maps_ctx(m, dtype, 1, max_len=704, page_size=16), [x], cuts, dtype, D)
+        got = _run_mixer(part, _maps_ctx(part, dtype, 1, max_len=704, page_size=16), [x], cuts, dtype, D)
         _close(got[0][-1], want[-1], dtype, f"key {back} back among {n}, map {which}, {len(cuts)} steps", b16=4e-2)
 
 
@@ -431,7 +440,7 @@ def test_query_temperature_steps_at_block_ends():
     assert px.query_temperature(17, 2.5, 8, F).tolist() == [1.0] * 7 + [1 + 2.5 * math.log(2)] * 8 + [1 + 2.5 * math.log(3)] * 2
     part = _maps_part(D, m, w, torch.float32)
     for cuts in ([[n]], [[7], [1], [1], [6], [2], [23]], [[1]] * n):
-        got = _run_mixer(part, _maps_ctx(m, torch.float32, 1), [x], cuts, torch.float32, D)
+        got = _run_mixer(part, _maps_ctx(part, torch.float32, 1), [x], cuts, torch.float32, D)
         _close(got[0], want, torch.float32, f"temperature, {len(cuts)} steps")
 
 
@@ -497,7 +506,7 @@ def test_requests_in_one_batch_equal_each_alone(dtype):
     fast = dict(MAPS, dim=32, vdim=64)
     fast_part, maps_part = (_maps_part(D, m, _maps_weights(D, m, g), dtype) for m in (fast, MAPS))
     delta_part = _delta_part(D, DELTA, _delta_weights(D, DELTA, g), dtype)
-    for part, ctx_of in ((maps_part, lambda n: _maps_ctx(MAPS, dtype, n)), (fast_part, lambda n: _maps_ctx(fast, dtype, n)),
+    for part, ctx_of in ((maps_part, lambda n: _maps_ctx(maps_part, dtype, n)), (fast_part, lambda n: _maps_ctx(fast_part, dtype, n)),
                          (delta_part, lambda n: StateCtx(dtype, n, state_floats=delta_part.state_need().shape[0]))):
         inputs = [_bf(torch.randn(n, D, generator=g)) for n in (33, 5, 12)]
         together = _run_mixer(part, ctx_of(3), inputs, [[20, 1, 3], [1, 1, 2], [12, 3, 7]], dtype, D)
