@@ -71,7 +71,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
                                const int* __restrict__ row_req, const int* __restrict__ positions,
                                const int* __restrict__ block_tables, int table_stride, int H, int Hkv, int hd,
                                int page_size, float scale, int window, int sink,
-                               const float* __restrict__ gate, int gate_ld, int gate_off, float out_scale) {
+                               const float* __restrict__ gate, int gate_ld, int gate_off, int gate_dims, float out_scale) {
     pdl_prologue();
     __shared__ float s_q[kMaxHeadDim];
     __shared__ float s_acc[kAttWarps][kMaxHeadDim];
@@ -146,14 +146,16 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_
         f[w] = (s_m[w] == -INFINITY) ? 0.f : expf(s_m[w] - M);
         L += s_l[w] * f[w];
     }
-    // an output gate per head: sigmoid of a 32-bit number of the token's row of ``gate``
+    // an output gate per head (or per value, with gate_dims): sigmoid of a 32-bit number of the token's row of ``gate``
     float mul = out_scale;
-    if (gate) mul *= 1.0f / (1.0f + expf(-gate[static_cast<size_t>(t) * gate_ld + gate_off + h]));
+    if (gate && !gate_dims) mul *= 1.0f / (1.0f + expf(-gate[static_cast<size_t>(t) * gate_ld + gate_off + h]));
+    const float* gz = gate_dims ? gate + static_cast<size_t>(t) * gate_ld + gate_off + static_cast<size_t>(h) * gate_dims : nullptr;
     for (int d = threadIdx.x; d < hd; d += blockDim.x) {
         float o = 0.f;
 #pragma unroll
         for (int w = 0; w < kAttWarps; ++w) o += s_acc[w][d] * f[w];
         o /= L;
+        if (gz) o *= sigmoid_f(gz[d]);
         out[(static_cast<size_t>(t) * H + h) * hd + d] = from_float<T>(gate || out_scale != 1.0f ? o * mul : o);
     }
 }
@@ -168,7 +170,7 @@ extern "C" int gi_attention_generic_supported(int hd) { return hd >= 1 && hd <= 
 static int gi_attention_generic_impl(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype,
                                     const int* row_req, const int* positions, const int* block_tables,
                                     int table_stride, int T, int H, int Hkv, int hd, int page_size, float scale,
-                                    int window, int sink, const float* gate, int gate_ld, int gate_off, float out_scale,
+                                    int window, int sink, const float* gate, int gate_ld, int gate_off, int gate_dims, float out_scale,
                                     void* stream) {
     if (T == 0) return 0;
     GI_REQUIRE(T > 0 && H > 0 && Hkv > 0 && page_size > 0, "attention: sizes must be positive");
@@ -181,12 +183,12 @@ static int gi_attention_generic_impl(const void* q, const void* k_cache, const v
         launch_kernel((paged_attention_generic_kernel<float>), dim3(grid), dim3(kAttWarps * 32), 0, st, 
             static_cast<const float*>(q), static_cast<const float*>(k_cache), static_cast<const float*>(v_cache),
             static_cast<float*>(out), row_req, positions, block_tables, table_stride, H, Hkv, hd, page_size, scale,
-            window, sink, gate, gate_ld, gate_off, out_scale);
+            window, sink, gate, gate_ld, gate_off, gate_dims, out_scale);
     } else if (dtype == kBF16) {
         launch_kernel((paged_attention_generic_kernel<__nv_bfloat16>), dim3(grid), dim3(kAttWarps * 32), 0, st, 
             static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),
             static_cast<const __nv_bfloat16*>(v_cache), static_cast<__nv_bfloat16*>(out), row_req, positions,
-            block_tables, table_stride, H, Hkv, hd, page_size, scale, window, sink, gate, gate_ld, gate_off, out_scale);
+            block_tables, table_stride, H, Hkv, hd, page_size, scale, window, sink, gate, gate_ld, gate_off, gate_dims, out_scale);
     } else {
         GI_REQUIRE(false, "attention: unsupported dtype code %d", dtype);
     }
@@ -195,6 +197,6 @@ static int gi_attention_generic_impl(const void* q, const void* k_cache, const v
 
 // The exported names: each runs its implementation above and, while a launch program is recorded, leaves a copy of
 // its arguments in the program (common.cuh).
-extern "C" int gi_attention_generic(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype, const int* row_req, const int* positions, const int* block_tables, int table_stride, int T, int H, int Hkv, int hd, int page_size, float scale, int window, int sink, const float* gate, int gate_ld, int gate_off, float out_scale, void* stream) {
-    return gi::dispatch(gi_attention_generic_impl, q, k_cache, v_cache, out, dtype, row_req, positions, block_tables, table_stride, T, H, Hkv, hd, page_size, scale, window, sink, gate, gate_ld, gate_off, out_scale, stream);
+extern "C" int gi_attention_generic(const void* q, const void* k_cache, const void* v_cache, void* out, int dtype, const int* row_req, const int* positions, const int* block_tables, int table_stride, int T, int H, int Hkv, int hd, int page_size, float scale, int window, int sink, const float* gate, int gate_ld, int gate_off, int gate_dims, float out_scale, void* stream) {
+    return gi::dispatch(gi_attention_generic_impl, q, k_cache, v_cache, out, dtype, row_req, positions, block_tables, table_stride, T, H, Hkv, hd, page_size, scale, window, sink, gate, gate_ld, gate_off, gate_dims, out_scale, stream);
 }

@@ -621,6 +621,13 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                 __nv_bfloat16* dst = out + (static_cast<size_t>(ci.t) * H + ci.g * G + row) * HD + (lane & 3) * 2;
                 if (!ep.plain()) {
                     const float f = att_finish(ep, l[r], m[r], ci.t, ci.g * G + row);
+                    if (ep.gate_dims) {
+                        const float* gz = att_gate_row(ep, ci.t, ci.g * G + row) + (lane & 3) * 2;
+#pragma unroll
+                        for (int n = 0; n < HD / 8; ++n)
+                            *reinterpret_cast<__nv_bfloat162*>(dst + n * 8) = __floats2bfloat162_rn(o[n][2 * r] * f * sigmoid_f(gz[n * 8]), o[n][2 * r + 1] * f * sigmoid_f(gz[n * 8 + 1]));
+                        continue;
+                    }
 #pragma unroll
                     for (int n = 0; n < HD / 8; ++n)
                         *reinterpret_cast<__nv_bfloat162*>(dst + n * 8) = __floats2bfloat162_rn(o[n][2 * r] * f, o[n][2 * r + 1] * f);
@@ -715,10 +722,12 @@ attention_combine_kernel(const float* __restrict__ part_o, const float* __restri
 #pragma unroll
     for (int w = 0; w < kCombineWarps; ++w) total += s_l[w];
     const float f = ep.plain() ? 0.f : att_finish(ep, total, M, t, h);
+    const float* gz = att_gate_row(ep, t, h);
     for (int d = threadIdx.x; d < HD; d += kCombineWarps * 32) {
         float o = 0.f;
 #pragma unroll
         for (int w = 0; w < kCombineWarps; ++w) o += s_acc[w][d];
+        if (gz) o *= sigmoid_f(gz[d]);
         out[(static_cast<size_t>(t) * H + h) * HD + d] = __float2bfloat16_rn(ep.plain() ? o / total : o * f);
     }
 }
@@ -1004,6 +1013,13 @@ attention_prefill_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __
         const int tok = row / G, hh = row % G;
         const float inv = ep.plain() ? 1.0f / l[r] : att_finish(ep, l[r], m[r], t0 + tok, g * G + hh);
         __nv_bfloat16* dst = out + (static_cast<size_t>(t0 + tok) * H + g * G + hh) * HD + (lane & 3) * 2;
+        if (ep.gate_dims) {
+            const float* gz = att_gate_row(ep, t0 + tok, g * G + hh) + (lane & 3) * 2;
+#pragma unroll
+            for (int n = 0; n < HD / 8; ++n)
+                *reinterpret_cast<__nv_bfloat162*>(dst + n * 8) = __floats2bfloat162_rn(o[n][2 * r] * inv * sigmoid_f(gz[n * 8]), o[n][2 * r + 1] * inv * sigmoid_f(gz[n * 8 + 1]));
+            continue;
+        }
 #pragma unroll
         for (int n = 0; n < HD / 8; ++n)
             *reinterpret_cast<__nv_bfloat162*>(dst + n * 8) = __floats2bfloat162_rn(o[n][2 * r] * inv, o[n][2 * r + 1] * inv);
@@ -1157,10 +1173,10 @@ static int gi_attention_decode_impl(const void* q, const void* k_cache, const vo
                                    int n_rows, const int* row_req, const int* positions, const int* block_tables,
                                    int table_stride, int H, int Hkv, int hd, int page_size, float scale, int window,
                                    float* part_o, float* part_ml, int max_chunks, int n_chunks, long long n_pages,
-                                   void* status, int sink, const float* gate, int gate_ld, int gate_off, float out_scale,
+                                   void* status, int sink, const float* gate, int gate_ld, int gate_off, int gate_dims, float out_scale,
                                    float softcap, void* stream) {
     if (n_rows == 0) return 0;
-    const AttEpilogue ep{sink, gate, gate_ld, gate_off, out_scale, softcap > 0.f ? softcap : 0.f};
+    const AttEpilogue ep{sink, gate, gate_ld, gate_off, gate_dims, out_scale, softcap > 0.f ? softcap : 0.f};
     GI_REQUIRE(gi_attention_fast_supported(hd, H, Hkv), "attention_decode: head size %d with %d/%d heads is not built", hd, H, Hkv);
     GI_REQUIRE(n_chunks >= 1 && n_chunks <= max_chunks, "attention_decode: %d chunks exceed the workspace's %d", n_chunks, max_chunks);
     GI_REQUIRE(n_rows <= 65535 && Hkv <= 65535, "attention_decode: grid too large");
@@ -1197,10 +1213,10 @@ static int gi_attention_decode_impl(const void* q, const void* k_cache, const vo
 static int gi_attention_prefill_impl(const void* q, const void* k_cache, const void* v_cache, void* out, const int* work,
                                     int n_work, const int* positions, const int* block_tables, int table_stride, int H,
                                     int Hkv, int hd, int page_size, float scale, int window, long long n_pages,
-                                    void* status, int sink, const float* gate, int gate_ld, int gate_off, float out_scale,
+                                    void* status, int sink, const float* gate, int gate_ld, int gate_off, int gate_dims, float out_scale,
                                     void* stream) {
     if (n_work == 0) return 0;
-    const AttEpilogue ep{sink, gate, gate_ld, gate_off, out_scale};
+    const AttEpilogue ep{sink, gate, gate_ld, gate_off, gate_dims, out_scale};
     GI_REQUIRE(gi_attention_fast_supported(hd, H, Hkv), "attention_prefill: head size %d with %d/%d heads is not built", hd, H, Hkv);
     GI_REQUIRE(n_work <= 65535, "attention_prefill: %d work items exceed the grid limit 65535", n_work);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
@@ -1229,10 +1245,10 @@ static int gi_attention_prefill_impl(const void* q, const void* k_cache, const v
 
 // The exported names: each runs its implementation above and, while a launch program is recorded, leaves a copy of
 // its arguments in the program (common.cuh).
-extern "C" int gi_attention_decode(const void* q, const void* k_cache, const void* v_cache, void* out, const int* rows, int n_rows, const int* row_req, const int* positions, const int* block_tables, int table_stride, int H, int Hkv, int hd, int page_size, float scale, int window, float* part_o, float* part_ml, int max_chunks, int n_chunks, long long n_pages, void* status, int sink, const float* gate, int gate_ld, int gate_off, float out_scale, float softcap, void* stream) {
-    return gi::dispatch(gi_attention_decode_impl, q, k_cache, v_cache, out, rows, n_rows, row_req, positions, block_tables, table_stride, H, Hkv, hd, page_size, scale, window, part_o, part_ml, max_chunks, n_chunks, n_pages, status, sink, gate, gate_ld, gate_off, out_scale, softcap, stream);
+extern "C" int gi_attention_decode(const void* q, const void* k_cache, const void* v_cache, void* out, const int* rows, int n_rows, const int* row_req, const int* positions, const int* block_tables, int table_stride, int H, int Hkv, int hd, int page_size, float scale, int window, float* part_o, float* part_ml, int max_chunks, int n_chunks, long long n_pages, void* status, int sink, const float* gate, int gate_ld, int gate_off, int gate_dims, float out_scale, float softcap, void* stream) {
+    return gi::dispatch(gi_attention_decode_impl, q, k_cache, v_cache, out, rows, n_rows, row_req, positions, block_tables, table_stride, H, Hkv, hd, page_size, scale, window, part_o, part_ml, max_chunks, n_chunks, n_pages, status, sink, gate, gate_ld, gate_off, gate_dims, out_scale, softcap, stream);
 }
 
-extern "C" int gi_attention_prefill(const void* q, const void* k_cache, const void* v_cache, void* out, const int* work, int n_work, const int* positions, const int* block_tables, int table_stride, int H, int Hkv, int hd, int page_size, float scale, int window, long long n_pages, void* status, int sink, const float* gate, int gate_ld, int gate_off, float out_scale, void* stream) {
-    return gi::dispatch(gi_attention_prefill_impl, q, k_cache, v_cache, out, work, n_work, positions, block_tables, table_stride, H, Hkv, hd, page_size, scale, window, n_pages, status, sink, gate, gate_ld, gate_off, out_scale, stream);
+extern "C" int gi_attention_prefill(const void* q, const void* k_cache, const void* v_cache, void* out, const int* work, int n_work, const int* positions, const int* block_tables, int table_stride, int H, int Hkv, int hd, int page_size, float scale, int window, long long n_pages, void* status, int sink, const float* gate, int gate_ld, int gate_off, int gate_dims, float out_scale, void* stream) {
+    return gi::dispatch(gi_attention_prefill_impl, q, k_cache, v_cache, out, work, n_work, positions, block_tables, table_stride, H, Hkv, hd, page_size, scale, window, n_pages, status, sink, gate, gate_ld, gate_off, gate_dims, out_scale, stream);
 }

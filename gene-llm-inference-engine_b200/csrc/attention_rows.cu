@@ -9,6 +9,7 @@
 //   slopes   [H] or null: slope_h * (P - j) is taken off the score of key j (a bias that grows with the distance)
 //   sinks    [H] or null: the softmax's denominator also holds exp(sinks_h), a term without key or value
 //   softcap  c > 0: the scaled score s becomes c tanh(s / c) before bias and softmax
+//   gate     [T, ldg] or null: value d of head h's output is multiplied by sigmoid(gate[t, gate_off + h * vd + d])
 //   values   a width ``vd`` of their own; they may lie in pages of their own or be the first vd columns of the key
 //            rows (``v_row`` is the length of the rows they lie in), which serves attention over a shared latent whose
 //            keys are [latent, rotated part] and whose values are the latent itself
@@ -38,11 +39,16 @@ struct RowsArgs {
     int H, Hkv, hd, vd, v_row, page_size;
     float scale; float softcap; int window, chunk;
     const float* slopes; const float* sinks;
+    const float* gate; int ldg, gate_off;          // 32-bit gate values in a row of the token, laid out as the output (else null)
     int heads_per_block;                           // query heads of one key/value head that a block takes
     int ks;                                        // row length of the key tile in shared memory (elements)
     int alias;                                     // the values are the first vd columns of the key rows
 };
 
+// The gate's values of head h of row t, from value dimension 0 on.
+__device__ __forceinline__ const float* gate_row(const RowsArgs& a, int t, int h) {
+    return a.gate ? a.gate + static_cast<size_t>(t) * a.ldg + a.gate_off + static_cast<size_t>(h) * a.vd : nullptr;
+}
 __device__ __forceinline__ float capped(float score, float cap) { return cap > 0.f ? cap * tanhf(score / cap) : score; }
 
 // HPW: query heads per warp; VI: value dimensions per lane (vd <= 32 * VI).
@@ -178,11 +184,13 @@ attention_rows_kernel(const RowsArgs a) {
         }
         const float mul = f / L;
         const size_t o = static_cast<size_t>(t) * a.ldo + static_cast<size_t>(h) * a.vd;
+        const float* gz = gate_row(a, t, h);
 #pragma unroll
         for (int i = 0; i < VI; ++i) {
             const int d = lane + 32 * i;
             if (d < a.vd) {
-                const float v = acc[hh][i] * mul;
+                float v = acc[hh][i] * mul;
+                if (gz) v *= sigmoid_f(gz[d]);
                 if (a.out_is_f32) static_cast<float*>(a.out)[o + d] = v;
                 else static_cast<__nv_bfloat16*>(a.out)[o + d] = __float2bfloat16_rn(v);
             }
@@ -510,10 +518,13 @@ attention_rows_mma_kernel(const RowsArgs a, const RowTiles rt) {
         }
         const float mul = f / L;
         const size_t ob = static_cast<size_t>(tr.row0 + tr.token(r)) * a.ldo + static_cast<size_t>(head) * a.vd + v0 + 2 * tq;
+        const float* gz = gate_row(a, tr.row0 + tr.token(r), head);
+        if (gz) gz += v0 + 2 * tq;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             if (i < nv) {
-                const float x0 = o[i][2 * h] * mul, x1 = o[i][2 * h + 1] * mul;
+                float x0 = o[i][2 * h] * mul, x1 = o[i][2 * h + 1] * mul;
+                if (gz) { x0 *= sigmoid_f(gz[i * 8]); x1 *= sigmoid_f(gz[i * 8 + 1]); }
                 if (a.out_is_f32) *reinterpret_cast<float2*>(static_cast<float*>(a.out) + ob + i * 8) = make_float2(x0, x1);
                 else *reinterpret_cast<uint32_t*>(static_cast<bf*>(a.out) + ob + i * 8) = rows_pack(x0, x1);
             }
@@ -554,11 +565,13 @@ attention_rows_merge_kernel(const RowsArgs a, const RowTiles rt) {
     }
     __syncthreads();
     const size_t ob = static_cast<size_t>(tr.row0 + tr.token(r)) * a.ldo + static_cast<size_t>(head) * a.vd;
+    const float* gz = gate_row(a, tr.row0 + tr.token(r), head);
     for (int d = threadIdx.x; d < a.vd; d += 128) {
         float v = 0.f;
 #pragma unroll 4
         for (int s = 0; s < rt.splits; ++s) v = fmaf(row[s * stride + d], s_w[s], v);
         v *= s_inv;
+        if (gz) v *= sigmoid_f(gz[d]);
         if (a.out_is_f32) static_cast<float*>(a.out)[ob + d] = v;
         else static_cast<__nv_bfloat16*>(a.out)[ob + d] = __float2bfloat16_rn(v);
     }
@@ -652,7 +665,7 @@ static int gi_attention_rows_impl(const void* q, int q_dtype, int ldq, const voi
                                  void* out, int out_dtype, int ldo, const int* row_req, const int* positions,
                                  const int* block_tables, int table_stride, int T, int H, int Hkv, int hd, int vd, int v_row,
                                  int values_in_keys, int page_size, float scale, float softcap, int window, int chunk, const float* slopes,
-                                 const float* sinks, const int* tile_list, int list_kind, int n_tiles, int splits, float* workspace,
+                                 const float* sinks, const float* gate, int ldg, int gate_off, const int* tile_list, int list_kind, int n_tiles, int splits, float* workspace,
                                  long long workspace_floats, void* stream) {
     if (T == 0 || (list_kind != 0 && n_tiles == 0)) return 0;
     GI_REQUIRE(T > 0 && H > 0 && Hkv > 0 && page_size > 0, "attention_rows: sizes must be positive");
@@ -672,6 +685,8 @@ static int gi_attention_rows_impl(const void* q, int q_dtype, int ldq, const voi
     a.row_req = row_req; a.positions = positions; a.block_tables = block_tables; a.table_stride = table_stride;
     a.H = H; a.Hkv = Hkv; a.hd = hd; a.vd = vd; a.v_row = v_row; a.page_size = page_size;
     a.scale = scale; a.softcap = softcap; a.window = window; a.chunk = chunk; a.slopes = slopes; a.sinks = sinks;
+    GI_REQUIRE(gate == nullptr || (gate_off >= 0 && gate_off + static_cast<long long>(H) * vd <= ldg), "attention_rows: the gate's columns lie outside its rows");
+    a.gate = gate; a.ldg = ldg; a.gate_off = gate_off;
     a.alias = values_in_keys ? 1 : 0;
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     // bfloat16 cache and sizes in whole MMA tiles: the tensor-core form (tiles of rows from the caller's list, or a row each)
@@ -723,9 +738,9 @@ extern "C" int gi_attention_rows(const void* q, int q_dtype, int ldq, const void
                                  void* out, int out_dtype, int ldo, const int* row_req, const int* positions,
                                  const int* block_tables, int table_stride, int T, int H, int Hkv, int hd, int vd, int v_row,
                                  int values_in_keys, int page_size, float scale, float softcap, int window, int chunk, const float* slopes,
-                                 const float* sinks, const int* tile_list, int list_kind, int n_tiles, int splits, float* workspace,
+                                 const float* sinks, const float* gate, int ldg, int gate_off, const int* tile_list, int list_kind, int n_tiles, int splits, float* workspace,
                                  long long workspace_floats, void* stream) {
     return gi::dispatch(gi_attention_rows_impl, q, q_dtype, ldq, k_cache, v_cache, cache_dtype, out, out_dtype, ldo, row_req,
                         positions, block_tables, table_stride, T, H, Hkv, hd, vd, v_row, values_in_keys, page_size, scale, softcap, window,
-                        chunk, slopes, sinks, tile_list, list_kind, n_tiles, splits, workspace, workspace_floats, stream);
+                        chunk, slopes, sinks, gate, ldg, gate_off, tile_list, list_kind, n_tiles, splits, workspace, workspace_floats, stream);
 }

@@ -519,12 +519,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
             // (a row beyond the tile's rows has seen no key: its sum is 0 and nothing of it is stored)
             const float inv = (ep.plain() || !row_valid) ? 1.0f / l : att_finish(ep, l, m_ref, t0 + tok, g * G + hh);
             __nv_bfloat16* dst = out + (static_cast<size_t>(t0 + tok) * H + g * G + hh) * HD;
+            const float* gz = row_valid ? att_gate_row(ep, t0 + tok, g * G + hh) : nullptr;
 #pragma unroll 1
             for (int c = 0; c < HD / 32; ++c) {
                 uint32_t ov[32];
                 tmem_ld32(tmem_o + lane_addr + c * 32, ov);
                 tmem_ld_wait();
                 if (row_valid) {
+                    if (gz) {
+#pragma unroll
+                        for (int e = 0; e < 32; ++e) ov[e] = __float_as_uint(__uint_as_float(ov[e]) * sigmoid_f(gz[c * 32 + e]));
+                    }
 #pragma unroll
                     for (int q4 = 0; q4 < 4; ++q4) {
                         uint32_t w[4];
@@ -596,10 +601,10 @@ extern "C" int gi_attention_prefill_tc_supported(int hd, int H, int Hkv, int pag
 static int gi_attention_prefill_tc_impl(const void* q, const void* k_cache, const void* v_cache, void* out, const int* work,
                                        int n_work, const int* positions, const int* block_tables, int table_stride, int H,
                                        int Hkv, int hd, int page_size, float scale, int window, long long n_pages,
-                                       void* status, int sink, const float* gate, int gate_ld, int gate_off, float out_scale,
+                                       void* status, int sink, const float* gate, int gate_ld, int gate_off, int gate_dims, float out_scale,
                                        float softcap, void* stream) {
     if (n_work == 0) return 0;
-    const AttEpilogue ep{sink, gate, gate_ld, gate_off, out_scale};
+    const AttEpilogue ep{sink, gate, gate_ld, gate_off, gate_dims, out_scale};
     GI_REQUIRE(gi_attention_prefill_tc_supported(hd, H, Hkv, page_size), "attention_prefill_tc: shape not supported");
     GI_REQUIRE(status != nullptr, "attention_prefill_tc: a status word is required");
     GI_REQUIRE(n_work <= 65535, "attention_prefill_tc: %d work items exceed the grid limit 65535", n_work);
@@ -620,6 +625,6 @@ static int gi_attention_prefill_tc_impl(const void* q, const void* k_cache, cons
 
 // The exported names: each runs its implementation above and, while a launch program is recorded, leaves a copy of
 // its arguments in the program (common.cuh).
-extern "C" int gi_attention_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out, const int* work, int n_work, const int* positions, const int* block_tables, int table_stride, int H, int Hkv, int hd, int page_size, float scale, int window, long long n_pages, void* status, int sink, const float* gate, int gate_ld, int gate_off, float out_scale, float softcap, void* stream) {
-    return gi::dispatch(gi_attention_prefill_tc_impl, q, k_cache, v_cache, out, work, n_work, positions, block_tables, table_stride, H, Hkv, hd, page_size, scale, window, n_pages, status, sink, gate, gate_ld, gate_off, out_scale, softcap, stream);
+extern "C" int gi_attention_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out, const int* work, int n_work, const int* positions, const int* block_tables, int table_stride, int H, int Hkv, int hd, int page_size, float scale, int window, long long n_pages, void* status, int sink, const float* gate, int gate_ld, int gate_off, int gate_dims, float out_scale, float softcap, void* stream) {
+    return gi::dispatch(gi_attention_prefill_tc_impl, q, k_cache, v_cache, out, work, n_work, positions, block_tables, table_stride, H, Hkv, hd, page_size, scale, window, n_pages, status, sink, gate, gate_ld, gate_off, gate_dims, out_scale, softcap, stream);
 }

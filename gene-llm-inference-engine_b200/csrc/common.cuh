@@ -89,11 +89,12 @@ __device__ __forceinline__ void pdl_prologue() { pdl_launch_dependents(); pdl_wa
 
 // What an attention kernel does to a finished row besides dividing by the softmax's sum: ``sink`` adds the weight of
 // one more key of score 0 (which has no value) to the sum, ``gate`` multiplies head h's output by
-// sigmoid(gate[t * gate_ld + gate_off + h]) (32-bit), ``out_scale`` by a constant. plain(): none of these.
+// sigmoid(gate[t * gate_ld + gate_off + h]) (32-bit) or, with ``gate_dims`` > 0, its value d by
+// sigmoid(gate[t * gate_ld + gate_off + h * gate_dims + d]), ``out_scale`` by a constant. plain(): none of these.
 struct AttEpilogue {
     int sink;
     const float* gate;
-    int gate_ld, gate_off;
+    int gate_ld, gate_off, gate_dims;
     float out_scale;
     float softcap = 0.f;      // c > 0: the scaled score s becomes c tanh(s / c) before the softmax (kernels that say they take it)
     __host__ __device__ bool plain() const { return !sink && gate == nullptr && out_scale == 1.0f; }
@@ -102,9 +103,14 @@ struct AttEpilogue {
 __device__ __forceinline__ float att_finish(const AttEpilogue& e, float l, float m_log2, int t, int h) {
     if (e.sink) l += exp2f(-m_log2);
     float f = e.out_scale / l;
-    if (e.gate) f *= 1.0f / (1.0f + expf(-e.gate[static_cast<size_t>(t) * e.gate_ld + e.gate_off + h]));
+    if (e.gate && !e.gate_dims) f *= 1.0f / (1.0f + expf(-e.gate[static_cast<size_t>(t) * e.gate_ld + e.gate_off + h]));
     return f;
 }
+// The gate's values of row (t, h) from dimension 0 on, where every value has one of its own; else null.
+__device__ __forceinline__ const float* att_gate_row(const AttEpilogue& e, int t, int h) {
+    return e.gate_dims ? e.gate + static_cast<size_t>(t) * e.gate_ld + e.gate_off + static_cast<size_t>(h) * e.gate_dims : nullptr;
+}
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // act(gate) * up of a gated feed-forward, 32-bit. 0 SiLU, 1 ReLU, 2 tanh-GELU; 3 ("capped swish"): the gate is capped from
 // above at `limit`, the up value clamped to [-limit, limit], and the result is gate * sigmoid(1.702 gate) * (up + 1).

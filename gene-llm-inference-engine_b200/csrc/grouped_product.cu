@@ -5,17 +5,21 @@
 //              W[h] = w + h * w_gs [N, K], out's columns o_off + h * o_gs .. + N; optionally ``tail`` more
 //              columns behind a head's K inputs are rotated by the row's position and copied behind its N outputs
 //              (queries of an attention over a shared latent: the plain part goes through the head's key matrix,
-//              the rotated part stays); optionally every output is multiplied by the sigmoid of a gate value of its own
-//              (32-bit, in a row of the token: the heads' outputs of a gated attention)
+//              the rotated part stays; pairs of neighbours or of the two halves); optionally every output is multiplied by
+//              the sigmoid of a gate value of its own, or of one of its head's (32-bit, in a row of the token: the heads'
+//              outputs of a gated attention)
 //     experts  rows are (token, choice) pairs sorted by expert: tile i belongs to expert tile_group[i], its rows are
 //              sorted_rows[16 i ..] (-1: none); the input row is pair / a_div, the output row the pair;
 //              gated: out = act(W_gate a) * (W_up a) with W[g] = [gate rows; up rows]; else optionally out = act(W a)
 //   route             per token: z = W_r x in 32-bit, s = sigmoid(z) or softmax(z) over all experts, the ``top`` experts by
-//                     s + correction; weights s, or s / (sum of the chosen s + 1e-20), times a constant
+//                     s + correction; weights s, or s / (sum of the chosen s + 1e-20), times a constant; optionally also
+//                     sigmoid(w_g x), one number per token (the gate of an expert that every token uses)
 //   route_align       buckets the pairs by expert into tiles of 16 rows (padding with -1), one block; for many rows
 //                     into tiles of 128, the token tiles of the tensor-core product that takes a matrix per tile
-//   gather_rows       a[r] = x[sorted_rows[r] / top] (zeros for padding): the rows in the tiles' order
-//   route_combine     y[t] += sum_k weight[t, k] * part[row of pair t * top + k] in the order of k
+//   gather_rows       a[r] = x[sorted_rows[r] / top] (zeros for padding): the rows in the tiles' order, optionally times
+//                     the pair's weight (where it scales what the expert reads)
+//   route_combine     y[t] += sum_k weight[t, k] * part[row of pair t * top + k] in the order of k (weights of 1 where they
+//                     scaled the experts' inputs), optionally plus gate[t] * more[t] (the gated expert of every token)
 //
 // Products run on the CUDA cores with 32-bit fused multiply-adds: the true 32-bit path, products of few rows (decoding,
 // where the weights stream once), the heads' matrices, and the bfloat16 path's fallback. Three forms: tiles of 16 x 64
@@ -38,16 +42,37 @@ struct GroupedArgs {
     int act; float act_limit;                                     // gated: a GateAct code and its limit
     int out_act;                                                  // not gated: a PlainAct code
     // rotated tail (heads form)
-    int tail; const float* freq; float amplitude; const int* positions;
-    // output gate (heads form): out *= sigmoid(gate[row, gate_off + h * N + n]), 32-bit (else null)
-    const float* gate; long long ldg; int gate_off;
+    int tail; const float* freq; float amplitude; int tail_interleaved; const int* positions;
+    // output gate (heads form): out *= sigmoid(gate[row, gate_off + h * gate_hs + n * gate_ns]), 32-bit (else null): a value
+    // per output (strides N, 1) or per head (1, 0)
+    const float* gate; long long ldg; int gate_off, gate_hs, gate_ns;
+    // experts form: what the products of a pair are multiplied with before the activation (the pair's weight when it scales
+    // what its expert reads), 32-bit by pair (else null)
+    const float* scales;
 };
+
+__device__ __forceinline__ float gp_gate_value(const GroupedArgs& p, int r, int g, int n) {
+    return p.gate[static_cast<size_t>(r) * p.ldg + p.gate_off + static_cast<size_t>(g) * p.gate_hs + static_cast<size_t>(n) * p.gate_ns];
+}
+
+// Pair pr of the rotated tail of row r, head g.
+template <typename TA>
+__device__ __forceinline__ void gp_rotate_pair(const GroupedArgs& p, const TA* tail_in, int r, int g, int pr) {
+    float sn, cs;
+    sincosf(static_cast<float>(p.positions[r]) * p.freq[pr], &sn, &cs);
+    sn *= p.amplitude; cs *= p.amplitude;
+    const int iu = p.tail_interleaved ? 2 * pr : pr, iv = p.tail_interleaved ? 2 * pr + 1 : pr + p.tail / 2;
+    const float u = to_float(tail_in[iu]), v = to_float(tail_in[iv]);
+    const size_t o = static_cast<size_t>(r) * p.ldo + p.o_off + static_cast<size_t>(g) * p.o_gs + p.N;
+    const float ru = u * cs - v * sn, rv = v * cs + u * sn;
+    if (p.out_is_f32) { static_cast<float*>(p.out)[o + iu] = ru; static_cast<float*>(p.out)[o + iv] = rv; }
+    else { static_cast<__nv_bfloat16*>(p.out)[o + iu] = __float2bfloat16_rn(ru); static_cast<__nv_bfloat16*>(p.out)[o + iv] = __float2bfloat16_rn(rv); }
+}
 
 // The element-wise sigmoid gate of the heads form, on output n of head g of row r.
 __device__ __forceinline__ float gp_gated(const GroupedArgs& p, float v, int r, int g, int n) {
     if (p.gate == nullptr) return v;
-    const float z = p.gate[static_cast<size_t>(r) * p.ldg + p.gate_off + static_cast<size_t>(g) * p.N + n];
-    return v * (1.0f / (1.0f + expf(-z)));
+    return v * sigmoid_f(gp_gate_value(p, r, g, n));
 }
 
 template <typename TA, typename TW, bool GATED>
@@ -81,15 +106,7 @@ grouped_product_kernel(const GroupedArgs p) {
             const int m = i / (p.tail / 2), pr = i % (p.tail / 2);
             const int r = s_row[m];
             if (r < 0) continue;
-            const TA* src = A + static_cast<size_t>(r) * p.lda + p.a_off + static_cast<size_t>(g) * p.a_gs + p.K + 2 * pr;
-            float sn, cs;
-            sincosf(static_cast<float>(p.positions[r]) * p.freq[pr], &sn, &cs);
-            sn *= p.amplitude; cs *= p.amplitude;
-            const float u = to_float(src[0]), v = to_float(src[1]);
-            const size_t o = static_cast<size_t>(r) * p.ldo + p.o_off + static_cast<size_t>(g) * p.o_gs + p.N + 2 * pr;
-            const float ru = u * cs - v * sn, rv = v * cs + u * sn;
-            if (p.out_is_f32) { static_cast<float*>(p.out)[o] = ru; static_cast<float*>(p.out)[o + 1] = rv; }
-            else { static_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16_rn(ru); static_cast<__nv_bfloat16*>(p.out)[o + 1] = __float2bfloat16_rn(rv); }
+            gp_rotate_pair(p, A + static_cast<size_t>(r) * p.lda + p.a_off + static_cast<size_t>(g) * p.a_gs + p.K, r, g, pr);
         }
     }
 
@@ -140,8 +157,9 @@ grouped_product_kernel(const GroupedArgs p) {
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tn + j;
             if (n >= p.N) continue;
-            float v = acc[i][j];
-            if (GATED) v = gated_value(v, acc_up[U * i][j], p.act, p.act_limit);
+            const float sc = p.scales ? p.scales[r] : 1.f;
+            float v = sc * acc[i][j];
+            if (GATED) v = gated_value(v, sc * acc_up[U * i][j], p.act, p.act_limit);
             else v = plain_value(v, p.out_act);
             v = gp_gated(p, v, r, g, n);
             const size_t o = static_cast<size_t>(r) * p.ldo + p.o_off + static_cast<size_t>(g) * p.o_gs + n;
@@ -229,7 +247,7 @@ grouped_rows_kernel(const GroupedArgs p) {
         if (p.gate != nullptr && lane < 4 * kGrFew) {
             const int gr = lane / kGrFew, gi_ = lane % kGrFew;
             if (gi_ < m_here && n_first + gr < p.N)
-                gate_z = p.gate[static_cast<size_t>(s_row[m0 + gi_]) * p.ldg + p.gate_off + static_cast<size_t>(g) * p.N + n_first + gr];
+                gate_z = gp_gate_value(p, s_row[m0 + gi_], g, n_first + gr);
         }
         for (int c = lane; c < pieces; c += 32) {
             float wv[4][8], uv[GATED ? 4 : 1][8];
@@ -268,8 +286,9 @@ grouped_rows_kernel(const GroupedArgs p) {
 #pragma unroll
             for (int i = 0; i < kGrFew; ++i) {
                 if (i < m_here && n_first + r < p.N) {
-                    float v = warp_sum(acc[r][i]);
-                    if (GATED) v = gated_value(v, warp_sum(acc_up[GATED ? r : 0][i]), p.act, p.act_limit);
+                    const float sc = p.scales ? p.scales[s_row[m0 + i]] : 1.f;
+                    float v = sc * warp_sum(acc[r][i]);
+                    if (GATED) v = gated_value(v, sc * warp_sum(acc_up[GATED ? r : 0][i]), p.act, p.act_limit);
                     else v = plain_value(v, p.out_act);
                     if (p.gate != nullptr) v *= 1.0f / (1.0f + expf(-__shfl_sync(0xffffffffu, gate_z, r * kGrFew + i)));
                     if (lane == 0) {
@@ -315,15 +334,7 @@ head_product64_kernel(const GroupedArgs p) {
             const int m = i / (p.tail / 2), pr = i % (p.tail / 2);
             const int r = row0 + m;
             if (r >= p.rows) continue;
-            const TA* src = A + static_cast<size_t>(r) * p.lda + p.K + 2 * pr;
-            float sn, cs;
-            sincosf(static_cast<float>(p.positions[r]) * p.freq[pr], &sn, &cs);
-            sn *= p.amplitude; cs *= p.amplitude;
-            const float u = to_float(src[0]), v = to_float(src[1]);
-            const size_t o = static_cast<size_t>(r) * p.ldo + p.o_off + static_cast<size_t>(g) * p.o_gs + p.N + 2 * pr;
-            const float ru = u * cs - v * sn, rv = v * cs + u * sn;
-            if (p.out_is_f32) { static_cast<float*>(p.out)[o] = ru; static_cast<float*>(p.out)[o + 1] = rv; }
-            else { static_cast<__nv_bfloat16*>(p.out)[o] = __float2bfloat16_rn(ru); static_cast<__nv_bfloat16*>(p.out)[o + 1] = __float2bfloat16_rn(rv); }
+            gp_rotate_pair(p, A + static_cast<size_t>(r) * p.lda + p.K, r, g, pr);
         }
     }
 
@@ -372,19 +383,22 @@ constexpr int kRouteMaxExperts = 1024;
 template <typename TX>
 __global__ void __launch_bounds__(128)
 route_kernel(const TX* __restrict__ x, int D, const float* __restrict__ w, const float* __restrict__ correction, int E, int top,
-             int softmax, int renormalise, float factor, int* __restrict__ ids, float* __restrict__ weights) {
+             int softmax, int renormalise, float factor, int* __restrict__ ids, float* __restrict__ weights,
+             const float* __restrict__ gate_w, float* __restrict__ gate_out) {
     pdl_prologue();
     extern __shared__ float s_x[];                 // [D]
     __shared__ float s_score[kRouteMaxExperts], s_choice[kRouteMaxExperts];
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     for (int d = threadIdx.x; d < D; d += 128) s_x[d] = to_float(x[static_cast<size_t>(t) * D + d]);
     __syncthreads();
-    for (int e = warp; e < E; e += 4) {
-        const float* row = w + static_cast<size_t>(e) * D;
+    for (int e = warp; e < E + (gate_w ? 1 : 0); e += 4) {
+        const float* row = e < E ? w + static_cast<size_t>(e) * D : gate_w;
         float z = 0.f;
         for (int d = lane; d < D; d += 32) z = fmaf(row[d], s_x[d], z);
         z = warp_sum(z);
-        if (lane == 0) {
+        if (e == E) {
+            if (lane == 0) gate_out[t] = sigmoid_f(z);
+        } else if (lane == 0) {
             const float s = softmax ? z : 1.0f / (1.0f + expf(-z));
             s_score[e] = s;
             s_choice[e] = s + (correction ? correction[e] : 0.f);
@@ -488,7 +502,7 @@ route_align_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __restr
 template <typename T>
 __global__ void __launch_bounds__(256)
 gather_rows_kernel(const T* __restrict__ x, int D, int a_div, const int* __restrict__ sorted_rows, const int* __restrict__ n_tiles,
-                   int tile_rows, T* __restrict__ out) {
+                   int tile_rows, const float* __restrict__ scales, T* __restrict__ out) {
     pdl_prologue();
     const int r = blockIdx.x;
     if (r >= *n_tiles * tile_rows) return;
@@ -499,6 +513,24 @@ gather_rows_kernel(const T* __restrict__ x, int D, int a_div, const int* __restr
         return;
     }
     const T* src = x + static_cast<size_t>(pair / a_div) * D;
+    if (scales) {
+        const float sc = scales[pair];
+        if (D % 8 == 0 && sizeof(T) == 2) {
+            for (int d = threadIdx.x; d < D / 8; d += 256) {
+                uint4 raw = reinterpret_cast<const uint4*>(src)[d];
+                __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const float2 f = __bfloat1622float2(h[i]);
+                    h[i] = __floats2bfloat162_rn(sc * f.x, sc * f.y);
+                }
+                reinterpret_cast<uint4*>(dst)[d] = raw;
+            }
+        } else {
+            for (int d = threadIdx.x; d < D; d += 256) dst[d] = from_float<T>(sc * to_float(src[d]));
+        }
+        return;
+    }
     if (D % 8 == 0 && sizeof(T) == 2) {
         for (int d = threadIdx.x; d < D / 8; d += 256) reinterpret_cast<uint4*>(dst)[d] = reinterpret_cast<const uint4*>(src)[d];
     } else {
@@ -508,7 +540,7 @@ gather_rows_kernel(const T* __restrict__ x, int D, int a_div, const int* __restr
 
 __global__ void __launch_bounds__(256)
 route_combine_kernel(const float* __restrict__ part, const float* __restrict__ weights, const int* __restrict__ pair_row,
-                     float* __restrict__ y, int D, int top, size_t total) {
+                     const float* __restrict__ more, const float* __restrict__ more_gate, float* __restrict__ y, int D, int top, size_t total) {
     pdl_prologue();
     const size_t i = static_cast<size_t>(blockIdx.x) * 256 + threadIdx.x;
     if (i >= total) return;
@@ -517,8 +549,9 @@ route_combine_kernel(const float* __restrict__ part, const float* __restrict__ w
     float v = y[i];
     for (int k = 0; k < top; ++k) {
         const size_t row = pair_row ? static_cast<size_t>(pair_row[t * top + k]) : t * top + k;
-        v = fmaf(weights[t * top + k], part[row * D + d], v);
+        v = fmaf(weights ? weights[t * top + k] : 1.f, part[row * D + d], v);
     }
+    if (more) v = fmaf(more_gate[t], more[i], v);
     y[i] = v;
 }
 
@@ -559,11 +592,11 @@ extern "C" int gi_grouped_tile_rows() { return kGpTM; }
 
 static int gi_head_product_impl(const void* a, int a_dtype, long long lda, int a_off, int a_gs, const void* w, int w_dtype,
                                 long long w_gs, void* out, int out_dtype, long long ldo, int o_off, int o_gs, int rows, int heads,
-                                int N, int K, int tail, const float* freq, float amplitude, const int* positions, const float* gate,
-                                long long ldg, int gate_off, void* stream) {
+                                int N, int K, int tail, const float* freq, float amplitude, int tail_interleaved, const int* positions, const float* gate,
+                                long long ldg, int gate_off, int gate_per_head, void* stream) {
     if (rows == 0) return 0;
     GI_REQUIRE(rows > 0 && heads > 0 && N > 0 && K > 0, "head_product: sizes must be positive");
-    GI_REQUIRE(gate == nullptr || (gate_off >= 0 && gate_off + static_cast<long long>(heads) * N <= ldg), "head_product: the gate's columns lie outside its rows");
+    GI_REQUIRE(gate == nullptr || (gate_off >= 0 && gate_off + static_cast<long long>(heads) * (gate_per_head ? 1 : N) <= ldg), "head_product: the gate's columns lie outside its rows");
     GI_REQUIRE(tail >= 0 && tail % 2 == 0 && (tail == 0 || (freq && positions)), "head_product: a rotated tail needs an even size, frequencies and positions");
     GI_REQUIRE(out_dtype == kF32 || out_dtype == kBF16, "head_product: unsupported output dtype");
     GroupedArgs p = {};
@@ -571,8 +604,8 @@ static int gi_head_product_impl(const void* a, int a_dtype, long long lda, int a
     p.w = w; p.w_gs = w_gs; p.ldw = K; p.up_off = 0;
     p.out = out; p.out_is_f32 = out_dtype == kF32; p.ldo = ldo; p.o_off = o_off; p.o_gs = o_gs;
     p.N = N; p.K = K; p.rows = rows; p.groups = heads;
-    p.tail = tail; p.freq = freq; p.amplitude = amplitude; p.positions = positions;
-    p.gate = gate; p.ldg = ldg; p.gate_off = gate_off;
+    p.tail = tail; p.freq = freq; p.amplitude = amplitude; p.tail_interleaved = tail_interleaved; p.positions = positions;
+    p.gate = gate; p.ldg = ldg; p.gate_off = gate_off; p.gate_hs = gate_per_head ? 1 : N; p.gate_ns = gate_per_head ? 0 : 1;
     const long long tiles = static_cast<long long>((rows + kGpTM - 1) / kGpTM) * heads;
     GI_REQUIRE(tiles <= 2147483647LL, "head_product: too many tiles");
     dim3 grid(static_cast<unsigned>(tiles), (N + kGpTN - 1) / kGpTN);
@@ -595,7 +628,7 @@ static int gi_head_product_impl(const void* a, int a_dtype, long long lda, int a
 }
 
 static int gi_expert_product_impl(const void* a, int a_dtype, long long lda, int a_div, const void* w, int w_dtype, long long w_gs,
-                                  int ldw, long long up_off, int gated, int act, float act_limit, void* out, int out_dtype, long long ldo,
+                                  int ldw, long long up_off, int gated, int act, float act_limit, const float* scales, void* out, int out_dtype, long long ldo,
                                   int N, int K, const int* tile_group, const int* sorted_rows, const int* n_tiles, int max_tiles,
                                   void* stream) {
     if (max_tiles == 0) return 0;
@@ -609,6 +642,7 @@ static int gi_expert_product_impl(const void* a, int a_dtype, long long lda, int
     p.N = N; p.K = K; p.groups = 1;
     p.tile_group = tile_group; p.sorted_rows = sorted_rows; p.n_tiles = n_tiles; p.act = gated ? act : 0; p.act_limit = act_limit;
     p.out_act = gated ? kPlainNone : act;
+    p.scales = scales;
     dim3 grid(max_tiles, (N + kGpTN - 1) / kGpTN);
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (rows_form_fits(p, a_dtype, w_dtype))
@@ -618,8 +652,9 @@ static int gi_expert_product_impl(const void* a, int a_dtype, long long lda, int
 
 static int gi_route_impl(const void* x, int x_dtype, int T, int D, const float* w, const float* correction, int E, int top,
                          int softmax, int renormalise, float factor, int* ids, float* weights, int* sorted_rows, int* tile_group, int* n_tiles, int max_tiles, int tile_rows,
-                         int* pair_row, void* stream) {
+                         int* pair_row, const float* gate_w, float* gate_out, void* stream) {
     if (T == 0) return 0;
+    GI_REQUIRE((gate_w == nullptr) == (gate_out == nullptr), "route: a gate needs its row and a place for its values");
     GI_REQUIRE(T > 0 && D > 0 && E > 0 && top > 0 && top <= E, "route: sizes must be positive and top at most the experts");
     GI_REQUIRE(E <= kRouteMaxExperts, "route: %d experts exceed %d", E, kRouteMaxExperts);
     GI_REQUIRE(static_cast<size_t>(D) * 4 <= 160 * 1024, "route: a row of %d values does not fit shared memory", D);
@@ -630,10 +665,10 @@ static int gi_route_impl(const void* x, int x_dtype, int T, int D, const float* 
     const size_t smem = static_cast<size_t>(D) * 4;
     if (x_dtype == kF32) {
         if (smem > 40 * 1024) cudaFuncSetAttribute(route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-        launch_kernel((route_kernel<float>), dim3(T), dim3(128), smem, st, static_cast<const float*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights);
+        launch_kernel((route_kernel<float>), dim3(T), dim3(128), smem, st, static_cast<const float*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights, gate_w, gate_out);
     } else if (x_dtype == kBF16) {
         if (smem > 40 * 1024) cudaFuncSetAttribute(route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-        launch_kernel((route_kernel<__nv_bfloat16>), dim3(T), dim3(128), smem, st, static_cast<const __nv_bfloat16*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights);
+        launch_kernel((route_kernel<__nv_bfloat16>), dim3(T), dim3(128), smem, st, static_cast<const __nv_bfloat16*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights, gate_w, gate_out);
     } else {
         GI_REQUIRE(false, "route: unsupported dtype code %d", x_dtype);
     }
@@ -660,50 +695,51 @@ static int gi_route_table_impl(const int* tokens, const int* feedback, const int
 }
 
 static int gi_gather_rows_impl(const void* x, int dtype, int D, int a_div, const int* sorted_rows, const int* n_tiles, int tile_rows,
-                               int max_rows, void* out, void* stream) {
+                               int max_rows, const float* scales, void* out, void* stream) {
     if (max_rows == 0) return 0;
     GI_REQUIRE(max_rows > 0 && D > 0 && a_div > 0 && tile_rows > 0, "gather_rows: sizes must be positive");
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (dtype == kBF16)
         launch_kernel((gather_rows_kernel<__nv_bfloat16>), dim3(max_rows), dim3(256), 0, st, static_cast<const __nv_bfloat16*>(x), D, a_div,
-                      sorted_rows, n_tiles, tile_rows, static_cast<__nv_bfloat16*>(out));
+                      sorted_rows, n_tiles, tile_rows, scales, static_cast<__nv_bfloat16*>(out));
     else if (dtype == kF32)
         launch_kernel((gather_rows_kernel<float>), dim3(max_rows), dim3(256), 0, st, static_cast<const float*>(x), D, a_div, sorted_rows,
-                      n_tiles, tile_rows, static_cast<float*>(out));
+                      n_tiles, tile_rows, scales, static_cast<float*>(out));
     else
         GI_REQUIRE(false, "gather_rows: unsupported dtype code %d", dtype);
     return check_launch("gather_rows");
 }
 
-static int gi_route_combine_impl(const float* part, const float* weights, const int* pair_row, float* y, int T, int D, int top, void* stream) {
+static int gi_route_combine_impl(const float* part, const float* weights, const int* pair_row, const float* more, const float* more_gate, float* y, int T, int D, int top, void* stream) {
     if (T == 0) return 0;
     GI_REQUIRE(T > 0 && D > 0 && top > 0, "route_combine: sizes must be positive");
+    GI_REQUIRE((more == nullptr) == (more_gate == nullptr), "route_combine: a gated part needs its gate");
     const size_t total = static_cast<size_t>(T) * D;
     launch_kernel(route_combine_kernel, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, static_cast<cudaStream_t>(stream),
-                  part, weights, pair_row, y, D, top, total);
+                  part, weights, pair_row, more, more_gate, y, D, top, total);
     return check_launch("route_combine");
 }
 
 extern "C" int gi_head_product(const void* a, int a_dtype, long long lda, int a_off, int a_gs, const void* w, int w_dtype,
                                long long w_gs, void* out, int out_dtype, long long ldo, int o_off, int o_gs, int rows, int heads,
-                               int N, int K, int tail, const float* freq, float amplitude, const int* positions, const float* gate,
-                               long long ldg, int gate_off, void* stream) {
+                               int N, int K, int tail, const float* freq, float amplitude, int tail_interleaved, const int* positions, const float* gate,
+                               long long ldg, int gate_off, int gate_per_head, void* stream) {
     return gi::dispatch(gi_head_product_impl, a, a_dtype, lda, a_off, a_gs, w, w_dtype, w_gs, out, out_dtype, ldo, o_off, o_gs, rows,
-                        heads, N, K, tail, freq, amplitude, positions, gate, ldg, gate_off, stream);
+                        heads, N, K, tail, freq, amplitude, tail_interleaved, positions, gate, ldg, gate_off, gate_per_head, stream);
 }
 
 extern "C" int gi_expert_product(const void* a, int a_dtype, long long lda, int a_div, const void* w, int w_dtype, long long w_gs,
-                                 int ldw, long long up_off, int gated, int act, float act_limit, void* out, int out_dtype, long long ldo, int N, int K,
+                                 int ldw, long long up_off, int gated, int act, float act_limit, const float* scales, void* out, int out_dtype, long long ldo, int N, int K,
                                  const int* tile_group, const int* sorted_rows, const int* n_tiles, int max_tiles, void* stream) {
-    return gi::dispatch(gi_expert_product_impl, a, a_dtype, lda, a_div, w, w_dtype, w_gs, ldw, up_off, gated, act, act_limit, out, out_dtype, ldo,
+    return gi::dispatch(gi_expert_product_impl, a, a_dtype, lda, a_div, w, w_dtype, w_gs, ldw, up_off, gated, act, act_limit, scales, out, out_dtype, ldo,
                         N, K, tile_group, sorted_rows, n_tiles, max_tiles, stream);
 }
 
 extern "C" int gi_route(const void* x, int x_dtype, int T, int D, const float* w, const float* correction, int E, int top,
                         int softmax, int renormalise, float factor, int* ids, float* weights, int* sorted_rows, int* tile_group, int* n_tiles, int max_tiles, int tile_rows, int* pair_row,
-                        void* stream) {
+                        const float* gate_w, float* gate_out, void* stream) {
     return gi::dispatch(gi_route_impl, x, x_dtype, T, D, w, correction, E, top, softmax, renormalise, factor, ids, weights, sorted_rows, tile_group, n_tiles,
-                        max_tiles, tile_rows, pair_row, stream);
+                        max_tiles, tile_rows, pair_row, gate_w, gate_out, stream);
 }
 
 extern "C" int gi_route_table(const int* tokens, const int* feedback, const int* table, int vocab, int T, int E, int top, int* ids,
@@ -714,10 +750,10 @@ extern "C" int gi_route_table(const int* tokens, const int* feedback, const int*
 }
 
 extern "C" int gi_gather_rows(const void* x, int dtype, int D, int a_div, const int* sorted_rows, const int* n_tiles, int tile_rows,
-                              int max_rows, void* out, void* stream) {
-    return gi::dispatch(gi_gather_rows_impl, x, dtype, D, a_div, sorted_rows, n_tiles, tile_rows, max_rows, out, stream);
+                              int max_rows, const float* scales, void* out, void* stream) {
+    return gi::dispatch(gi_gather_rows_impl, x, dtype, D, a_div, sorted_rows, n_tiles, tile_rows, max_rows, scales, out, stream);
 }
 
-extern "C" int gi_route_combine(const float* part, const float* weights, const int* pair_row, float* y, int T, int D, int top, void* stream) {
-    return gi::dispatch(gi_route_combine_impl, part, weights, pair_row, y, T, D, top, stream);
+extern "C" int gi_route_combine(const float* part, const float* weights, const int* pair_row, const float* more, const float* more_gate, float* y, int T, int D, int top, void* stream) {
+    return gi::dispatch(gi_route_combine_impl, part, weights, pair_row, more, more_gate, y, T, D, top, stream);
 }

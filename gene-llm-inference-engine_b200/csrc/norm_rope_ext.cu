@@ -6,7 +6,7 @@
 //   residual_norm   x = w * (acc / sqrt(mean(acc^2) + eps)) in 32-bit, in one pass also the next sublayer's
 //                   xn = x (compute dtype) and acc = alpha * x
 //   gated_act       out = act(gate) * up for act in {SiLU, ReLU, tanh-GELU, capped swish}, optionally with a bias on both
-//   norm_rope_store per token and head: optional unit-RMS norm with a weight shared by all heads, rotation of the
+//   norm_rope_store per token and head: an optional bias on every projected column, optional unit-RMS norm with a weight shared by all heads, rotation of the
 //                   first 2 * rot_half dimensions by angles position * freq[i] computed here in 32-bit (no table
 //                   of max_position rows), queries to q_out, keys to the token's page row; the values stored beside
 //                   them come from any column of the same input row (the keys as projected, for a design whose
@@ -17,7 +17,8 @@
 //                   adds its output to)
 //   latent_store    per token, from one row of 32-bit projections: a query latent brought to unit RMS and weighted,
 //                   to q_latent; a key/value latent likewise, into the first columns of the token's page row; a
-//                   rotated part shared by all heads (angles position * freq[i], cos and sin times a constant) behind it
+//                   rotated part shared by all heads (angles position * freq[i], cos and sin times a constant; pairs of
+//                   neighbours or of the two halves) behind it
 //
 // All arithmetic is 32-bit; only stores round. A row's result depends on that row only.
 #include "common.cuh"
@@ -123,7 +124,7 @@ constexpr int kNrsPairs = kNrsMaxHead / 64;
 
 template <typename T>
 __global__ void __launch_bounds__(kNrsWarps * 32)
-norm_rope_store_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, int v_off,
+norm_rope_store_kernel(const float* __restrict__ in, int ld, int q_off, int k_off, int v_off, const float* __restrict__ bias,
                        const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps,
                        const float* __restrict__ freq, int rot_half, int interleaved,
                        const int* __restrict__ positions, const int* __restrict__ row_req,
@@ -143,8 +144,9 @@ norm_rope_store_kernel(const float* __restrict__ in, int ld, int q_off, int k_of
     // [H * hd] and [Hkv * hd]; every block of the token takes the two sums over the whole row in the same order
     if (wide) {
         float sq = 0.f, sk = 0.f;
-        if (q_norm) for (int i = threadIdx.x; i < H * hd; i += kNrsWarps * 32) sq = fmaf(row[q_off + i], row[q_off + i], sq);
-        if (k_norm) for (int i = threadIdx.x; i < Hkv * hd; i += kNrsWarps * 32) sk = fmaf(row[k_off + i], row[k_off + i], sk);
+        auto value = [&](int c) { return bias ? row[c] + bias[c] : row[c]; };
+        if (q_norm) for (int i = threadIdx.x; i < H * hd; i += kNrsWarps * 32) sq = fmaf(value(q_off + i), value(q_off + i), sq);
+        if (k_norm) for (int i = threadIdx.x; i < Hkv * hd; i += kNrsWarps * 32) sk = fmaf(value(k_off + i), value(k_off + i), sk);
         sq = warp_sum(sq);
         sk = warp_sum(sk);
         if (lane == 0) { s_wide[0][warp] = sq; s_wide[1][warp] = sk; }
@@ -168,7 +170,9 @@ norm_rope_store_kernel(const float* __restrict__ in, int ld, int q_off, int k_of
     const int n_pairs = hd / 2;
     for (int head = blockIdx.y * kNrsWarps + warp; head < n_heads; head += kNrsWarps * gridDim.y) {
         const bool is_q = head < H;
-        const float* src = row + (is_q ? q_off + head * hd : k_off + (head - H) * hd);
+        const int col = is_q ? q_off + head * hd : k_off + (head - H) * hd;
+        const float* src = row + col;
+        const float* sbias = bias ? bias + col : nullptr;
         const float* nw = is_q ? q_norm : k_norm;
         if (nw && wide) nw += (is_q ? head : head - H) * hd;
         float va[kNrsPairs], vb[kNrsPairs];
@@ -187,6 +191,7 @@ norm_rope_store_kernel(const float* __restrict__ in, int ld, int q_off, int k_of
             const bool in_head = pr < n_pairs;
             va[u] = in_head ? src[ia[u]] : 0.f;
             vb[u] = in_head ? src[ib[u]] : 0.f;
+            if (sbias && in_head) { va[u] += sbias[ia[u]]; vb[u] += sbias[ib[u]]; }
             ss = fmaf(va[u], va[u], ss);
             ss = fmaf(vb[u], vb[u], ss);
         }
@@ -194,9 +199,11 @@ norm_rope_store_kernel(const float* __restrict__ in, int ld, int q_off, int k_of
                       : k_cache + kv_base + static_cast<size_t>(head - H) * page_size * hd;
         if (!is_q) {
             // the values: copied from their columns as they are (the keys themselves where the design says so)
-            const float* vsrc = row + v_off + (head - H) * vd;
+            const int vcol = v_off + (head - H) * vd;
+            const float* vsrc = row + vcol;
+            const float* vbias = bias ? bias + vcol : nullptr;
             T* vdst = v_cache + v_base + static_cast<size_t>(head - H) * page_size * vd;
-            for (int d = lane; d < vd; d += 32) vdst[d] = from_float<T>(vsrc[d]);
+            for (int d = lane; d < vd; d += 32) vdst[d] = from_float<T>(vbias ? vsrc[d] + vbias[d] : vsrc[d]);
         }
         if (nw) {
             ss = warp_sum(ss);
@@ -250,7 +257,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 latent_store_kernel(const float* __restrict__ in, int ld, int q_off, int q_rank, const float* __restrict__ q_weight,
                     T* __restrict__ q_latent, int c_off, int rank, const float* __restrict__ c_weight, int r_off, int rot,
-                    const float* __restrict__ freq, float amplitude, float eps, const int* __restrict__ positions,
+                    const float* __restrict__ freq, float amplitude, int interleaved, float eps, const int* __restrict__ positions,
                     const int* __restrict__ row_req, const int* __restrict__ block_tables, int table_stride,
                     T* __restrict__ cache, int page_size, int write_cache) {
     pdl_prologue();
@@ -276,9 +283,10 @@ latent_store_kernel(const float* __restrict__ in, int ld, int q_off, int q_rank,
         float sn, cs;
         sincosf(static_cast<float>(pos) * freq[pr], &sn, &cs);
         sn *= amplitude; cs *= amplitude;
-        const float u = row[r_off + 2 * pr], v = row[r_off + 2 * pr + 1];
-        dst[rank + 2 * pr] = from_float<T>(u * cs - v * sn);
-        dst[rank + 2 * pr + 1] = from_float<T>(v * cs + u * sn);
+        const int iu = interleaved ? 2 * pr : pr, iv = interleaved ? 2 * pr + 1 : pr + rot / 2;
+        const float u = row[r_off + iu], v = row[r_off + iv];
+        dst[rank + iu] = from_float<T>(u * cs - v * sn);
+        dst[rank + iv] = from_float<T>(v * cs + u * sn);
     }
 }
 
@@ -337,7 +345,7 @@ static int gi_gated_act_impl(const float* gate_up, const float* bias, void* out,
     return check_launch("gated_act");
 }
 
-static int gi_norm_rope_store_impl(const float* in, int ld, int q_off, int k_off, int v_off, const float* q_norm,
+static int gi_norm_rope_store_impl(const float* in, int ld, int q_off, int k_off, int v_off, const float* bias, const float* q_norm,
                                    const float* k_norm, float eps, const float* freq, int rot_half, int interleaved,
                                    const int* positions, const int* row_req, const int* block_tables, int table_stride,
                                    void* q_out, void* k_cache, void* v_cache, int dtype, int T, int H, int Hkv, int hd,
@@ -354,12 +362,12 @@ static int gi_norm_rope_store_impl(const float* in, int ld, int q_off, int k_off
     // few rows (decoding): the heads of a token are spread over blocks; many rows: a block per token
     const unsigned head_blocks = T >= 256 ? 1u : static_cast<unsigned>(std::min((H + Hkv + kNrsWarps - 1) / kNrsWarps, 65535));
     if (dtype == kF32)
-        launch_kernel((norm_rope_store_kernel<float>), dim3(T, head_blocks), dim3(kNrsWarps * 32), 0, st, in, ld, q_off, k_off, v_off, q_norm,
+        launch_kernel((norm_rope_store_kernel<float>), dim3(T, head_blocks), dim3(kNrsWarps * 32), 0, st, in, ld, q_off, k_off, v_off, bias, q_norm,
                       k_norm, eps, freq, rot_half, interleaved, positions, row_req, block_tables, table_stride,
                       static_cast<float*>(q_out), static_cast<float*>(k_cache), static_cast<float*>(v_cache), H, Hkv, hd,
                       vd, page_size, write_kv, wide);
     else if (dtype == kBF16)
-        launch_kernel((norm_rope_store_kernel<__nv_bfloat16>), dim3(T, head_blocks), dim3(kNrsWarps * 32), 0, st, in, ld, q_off, k_off, v_off,
+        launch_kernel((norm_rope_store_kernel<__nv_bfloat16>), dim3(T, head_blocks), dim3(kNrsWarps * 32), 0, st, in, ld, q_off, k_off, v_off, bias,
                       q_norm, k_norm, eps, freq, rot_half, interleaved, positions, row_req, block_tables, table_stride,
                       static_cast<__nv_bfloat16*>(q_out), static_cast<__nv_bfloat16*>(k_cache),
                       static_cast<__nv_bfloat16*>(v_cache), H, Hkv, hd, vd, page_size, write_kv, wide);
@@ -380,8 +388,8 @@ extern "C" int gi_gated_act(const float* gate_up, const float* bias, void* out, 
     return gi::dispatch(gi_gated_act_impl, gate_up, bias, out, out_dtype, T, I, act, limit, stream);
 }
 
-extern "C" int gi_norm_rope_store(const float* in, int ld, int q_off, int k_off, int v_off, const float* q_norm, const float* k_norm, float eps, const float* freq, int rot_half, int interleaved, const int* positions, const int* row_req, const int* block_tables, int table_stride, void* q_out, void* k_cache, void* v_cache, int dtype, int T, int H, int Hkv, int hd, int vd, int page_size, int write_kv, int wide, void* stream) {
-    return gi::dispatch(gi_norm_rope_store_impl, in, ld, q_off, k_off, v_off, q_norm, k_norm, eps, freq, rot_half, interleaved, positions, row_req, block_tables, table_stride, q_out, k_cache, v_cache, dtype, T, H, Hkv, hd, vd, page_size, write_kv, wide, stream);
+extern "C" int gi_norm_rope_store(const float* in, int ld, int q_off, int k_off, int v_off, const float* bias, const float* q_norm, const float* k_norm, float eps, const float* freq, int rot_half, int interleaved, const int* positions, const int* row_req, const int* block_tables, int table_stride, void* q_out, void* k_cache, void* v_cache, int dtype, int T, int H, int Hkv, int hd, int vd, int page_size, int write_kv, int wide, void* stream) {
+    return gi::dispatch(gi_norm_rope_store_impl, in, ld, q_off, k_off, v_off, bias, q_norm, k_norm, eps, freq, rot_half, interleaved, positions, row_req, block_tables, table_stride, q_out, k_cache, v_cache, dtype, T, H, Hkv, hd, vd, page_size, write_kv, wide, stream);
 }
 
 static int gi_add_normed_impl(float* y, const float* weight, float* x, void* xn_out, int xn_dtype, int rows, int D, float eps,
@@ -397,7 +405,7 @@ static int gi_add_normed_impl(float* y, const float* weight, float* x, void* xn_
 }
 
 static int gi_latent_store_impl(const float* in, int ld, int q_off, int q_rank, const float* q_weight, void* q_latent, int c_off,
-                                int rank, const float* c_weight, int r_off, int rot, const float* freq, float amplitude, float eps,
+                                int rank, const float* c_weight, int r_off, int rot, const float* freq, float amplitude, int interleaved, float eps,
                                 const int* positions, const int* row_req, const int* block_tables, int table_stride, void* cache,
                                 int dtype, int T, int page_size, int write_cache, void* stream) {
     if (T == 0) return 0;
@@ -408,11 +416,11 @@ static int gi_latent_store_impl(const float* in, int ld, int q_off, int q_rank, 
     cudaStream_t st = static_cast<cudaStream_t>(stream);
     if (dtype == kF32)
         launch_kernel((latent_store_kernel<float>), dim3(T), dim3(256), 0, st, in, ld, q_off, q_rank, q_weight, static_cast<float*>(q_latent),
-                      c_off, rank, c_weight, r_off, rot, freq, amplitude, eps, positions, row_req, block_tables, table_stride,
+                      c_off, rank, c_weight, r_off, rot, freq, amplitude, interleaved, eps, positions, row_req, block_tables, table_stride,
                       static_cast<float*>(cache), page_size, write_cache);
     else if (dtype == kBF16)
         launch_kernel((latent_store_kernel<__nv_bfloat16>), dim3(T), dim3(256), 0, st, in, ld, q_off, q_rank, q_weight,
-                      static_cast<__nv_bfloat16*>(q_latent), c_off, rank, c_weight, r_off, rot, freq, amplitude, eps, positions, row_req,
+                      static_cast<__nv_bfloat16*>(q_latent), c_off, rank, c_weight, r_off, rot, freq, amplitude, interleaved, eps, positions, row_req,
                       block_tables, table_stride, static_cast<__nv_bfloat16*>(cache), page_size, write_cache);
     else
         GI_REQUIRE(false, "latent_store: unsupported dtype code %d", dtype);
@@ -423,6 +431,6 @@ extern "C" int gi_add_normed(float* y, const float* weight, float* x, void* xn_o
     return gi::dispatch(gi_add_normed_impl, y, weight, x, xn_out, xn_dtype, rows, D, eps, clear_y, stream);
 }
 
-extern "C" int gi_latent_store(const float* in, int ld, int q_off, int q_rank, const float* q_weight, void* q_latent, int c_off, int rank, const float* c_weight, int r_off, int rot, const float* freq, float amplitude, float eps, const int* positions, const int* row_req, const int* block_tables, int table_stride, void* cache, int dtype, int T, int page_size, int write_cache, void* stream) {
-    return gi::dispatch(gi_latent_store_impl, in, ld, q_off, q_rank, q_weight, q_latent, c_off, rank, c_weight, r_off, rot, freq, amplitude, eps, positions, row_req, block_tables, table_stride, cache, dtype, T, page_size, write_cache, stream);
+extern "C" int gi_latent_store(const float* in, int ld, int q_off, int q_rank, const float* q_weight, void* q_latent, int c_off, int rank, const float* c_weight, int r_off, int rot, const float* freq, float amplitude, int interleaved, float eps, const int* positions, const int* row_req, const int* block_tables, int table_stride, void* cache, int dtype, int T, int page_size, int write_cache, void* stream) {
+    return gi::dispatch(gi_latent_store_impl, in, ld, q_off, q_rank, q_weight, q_latent, c_off, rank, c_weight, r_off, rot, freq, amplitude, interleaved, eps, positions, row_req, block_tables, table_stride, cache, dtype, T, page_size, write_cache, stream);
 }

@@ -188,6 +188,12 @@ take_stream_kernel(float* __restrict__ x, const float* __restrict__ from, TOut* 
     }
 }
 
+__global__ void __launch_bounds__(256)
+add_stream_kernel(float* __restrict__ x, const float* __restrict__ more, size_t total) {
+    pdl_prologue();
+    for (size_t i = static_cast<size_t>(blockIdx.x) * 256 + threadIdx.x; i < total; i += static_cast<size_t>(gridDim.x) * 256) x[i] += more[i];
+}
+
 template <typename TOut, int VEC>
 __global__ void __launch_bounds__(256)
 depth_mix_kernel(float* __restrict__ x, float* __restrict__ y, const float* __restrict__ y_bias, float m, float* __restrict__ hist, int slots, int slot,
@@ -469,6 +475,13 @@ static int gi_take_stream_impl(float* x, const float* from, void* xn, int xn_dty
     return check_launch("take_stream");
 }
 
+static int gi_add_stream_impl(float* x, const float* more, long long total, void* stream) {
+    if (total == 0) return 0;
+    GI_REQUIRE(total > 0, "add_stream: the size must be positive");
+    launch_kernel(add_stream_kernel, dim3(grid_for(static_cast<size_t>(total))), dim3(256), 0, static_cast<cudaStream_t>(stream), x, more, static_cast<size_t>(total));
+    return check_launch("add_stream");
+}
+
 static int gi_plain_act_impl(const float* z, void* out, int out_dtype, long long total, int act, void* stream) {
     if (total == 0) return 0;
     GI_REQUIRE(total > 0 && act >= 0 && act < kPlainCount, "plain_act: unknown activation code %d", act);
@@ -486,6 +499,10 @@ extern "C" int gi_plain_act(const float* z, void* out, int out_dtype, long long 
 
 extern "C" int gi_layer_norm(const float* x, const int* rows, const float* weight, const float* bias, void* out, int out_dtype, int n, int D, float eps, void* stream) {
     return gi::dispatch(gi_layer_norm_impl, x, rows, weight, bias, out, out_dtype, n, D, eps, stream);
+}
+
+extern "C" int gi_add_stream(float* x, const float* more, long long total, void* stream) {
+    return gi::dispatch(gi_add_stream_impl, x, more, total, stream);
 }
 
 extern "C" int gi_take_stream(float* x, const float* from, void* xn, int xn_dtype, long long total, void* stream) {

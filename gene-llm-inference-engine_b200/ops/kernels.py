@@ -240,17 +240,18 @@ def norm_rope_store(proj: torch.Tensor, q_offset: int, k_offset: int, v_offset: 
                     k_norm: Optional[torch.Tensor], eps: float, freq: Optional[torch.Tensor], interleaved: bool,
                     positions: torch.Tensor, row_req: torch.Tensor, block_tables: torch.Tensor, q_out: torch.Tensor,
                     k_cache: torch.Tensor, v_cache: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int,
-                    page_size: int, write_kv: bool = True, value_dim: Optional[int] = None, wide_norm: bool = False) -> None:
+                    page_size: int, write_kv: bool = True, value_dim: Optional[int] = None, wide_norm: bool = False,
+                    bias: Optional[torch.Tensor] = None) -> None:
     """From the 32-bit projections ``proj`` [T, ld] (query heads from column q_offset, key heads from k_offset,
-    value heads from v_offset, which may be the keys' columns): per head an optional unit-RMS norm with the
+    value heads from v_offset, which may be the keys' columns; ``bias`` [ld]: added to every column as it is read): per head an optional unit-RMS norm with the
     shared weight ``q_norm`` / ``k_norm`` [hd] (``wide_norm``: one norm over all query heads' values together and one
     over all key heads', with weights [H*hd] and [Hkv*hd]), then the rotation of the first 2 * len(freq) dimensions by
     position * freq[i] (angles computed on the device in 32-bit), queries to ``q_out`` [T, H*hd], keys and
     values into the token's page row. ``value_dim``: the width of a value head when it is not the head size."""
     T, ld = proj.shape
     vd = head_dim if value_dim is None else int(value_dim)
-    if q_out.shape != (T, num_heads * head_dim):
-        raise KernelError("norm_rope_store: q_out must be [T, H*hd]")
+    if q_out.shape != (T, num_heads * head_dim) or (bias is not None and bias.numel() != ld):
+        raise KernelError("norm_rope_store: q_out must be [T, H*hd] (and the bias have a value per column)")
     if k_cache.dtype != q_out.dtype or v_cache.dtype != q_out.dtype:
         raise KernelError("norm_rope_store: q_out and the cache must have one dtype")
     if k_cache.shape[1:] != (num_kv_heads, page_size, head_dim) or v_cache.shape != (k_cache.shape[0], num_kv_heads, page_size, vd):
@@ -259,7 +260,7 @@ def norm_rope_store(proj: torch.Tensor, q_offset: int, k_offset: int, v_offset: 
         if w is not None and w.numel() != (heads * head_dim if wide_norm else head_dim):
             raise KernelError(f"norm_rope_store: {name} must have head_dim values (all heads' with wide_norm)")
     check(lib().gi_norm_rope_store(
-        _dev(proj, "proj", torch.float32), ld, int(q_offset), int(k_offset), int(v_offset),
+        _dev(proj, "proj", torch.float32), ld, int(q_offset), int(k_offset), int(v_offset), _opt(bias, "bias", torch.float32),
         _opt(q_norm, "q_norm", torch.float32), _opt(k_norm, "k_norm", torch.float32), float(eps),
         _opt(freq, "freq", torch.float32), 0 if freq is None else freq.numel(), int(interleaved),
         _dev(positions, "positions", torch.int32), _dev(row_req, "row_req", torch.int32),
@@ -413,12 +414,49 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out: t
           "layer_norm")
 
 
+def dynamic_tanh(x: torch.Tensor, alpha: float, weight: torch.Tensor, bias: torch.Tensor, out: torch.Tensor,
+                 rows: Optional[torch.Tensor] = None) -> None:
+    """out[r, :] = tanh(alpha * x[r, :]) * weight + bias of row r of x (of row rows[r] with ``rows``)."""
+    n, D = out.shape
+    if x.shape[1] != D or weight.numel() != D or bias.numel() != D:
+        raise KernelError("dynamic_tanh: shapes of x, weight, bias and out do not agree")
+    if (rows is None and x.shape[0] < n) or (rows is not None and rows.numel() != n):
+        raise KernelError("dynamic_tanh: rows and out do not agree")
+    check(lib().gi_dynamic_tanh(_dev(x, "x", torch.float32), _opt(rows, "rows", torch.int32), float(alpha), _dev(weight, "weight", torch.float32),
+                                _dev(bias, "bias", torch.float32), _dev(out, "out"), dtype_code(out.dtype), n, D, _stream()), "dynamic_tanh")
+
+
+def add_dynamic_tanh(y: torch.Tensor, norm, x: torch.Tensor, more: Optional[torch.Tensor] = None, next_norm=None,
+                     xn_out: Optional[torch.Tensor] = None, clear_y: bool = False) -> None:
+    """x += tanh(alpha * y) * weight + bias with ``norm`` = (alpha, weight [D], bias [D]), in 32-bit, plus ``more`` [T, D] when
+    given; optionally also xn_out = the ``next_norm`` of the new x in xn_out's dtype, and y = 0: the end of a sublayer whose
+    output is normed before it joins the stream, with what the next sublayer reads and adds to."""
+    n, D = y.shape
+    alpha, weight, bias = norm
+    next_alpha, next_weight, next_bias = next_norm if next_norm is not None else (0.0, None, None)
+    if x.shape != y.shape or weight.numel() != D or bias.numel() != D or (more is not None and more.shape != y.shape) or \
+            (xn_out is not None and (xn_out.shape != y.shape or next_norm is None or next_weight.numel() != D or next_bias.numel() != D)):
+        raise KernelError("add_dynamic_tanh: shapes do not agree (or xn_out comes without a norm)")
+    check(lib().gi_add_dynamic_tanh(_dev(y, "y", torch.float32), float(alpha), _dev(weight, "weight", torch.float32),
+                                    _dev(bias, "bias", torch.float32), _dev(x, "x", torch.float32), _opt(more, "more", torch.float32),
+                                    float(next_alpha), _opt(next_weight, "next weight", torch.float32), _opt(next_bias, "next bias", torch.float32),
+                                    0 if xn_out is None else _dev(xn_out, "xn_out"), F32 if xn_out is None else dtype_code(xn_out.dtype),
+                                    n, D, int(bool(clear_y)), _stream()), "add_dynamic_tanh")
+
+
 def take_stream(x: torch.Tensor, start: torch.Tensor, xn: torch.Tensor) -> None:
     """xn = x in xn's dtype and x = start, 32-bit: what a product that replaces the stream reads and adds to."""
     if start.shape != x.shape or xn.shape != x.shape:
         raise KernelError("take_stream: shapes do not agree")
     check(lib().gi_take_stream(_dev(x, "x", torch.float32), _dev(start, "start", torch.float32), _dev(xn, "xn"), dtype_code(xn.dtype),
                                x.numel(), _stream()), "take_stream")
+
+
+def add_stream(x: torch.Tensor, more: torch.Tensor) -> None:
+    """x += more, 32-bit."""
+    if more.shape != x.shape:
+        raise KernelError("add_stream: shapes do not agree")
+    check(lib().gi_add_stream(_dev(x, "x", torch.float32), _dev(more, "more", torch.float32), x.numel(), _stream()), "add_stream")
 
 
 def streams(X: torch.Tensor, single: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None, clear_y: bool = False,
@@ -447,12 +485,12 @@ def streams(X: torch.Tensor, single: Optional[torch.Tensor] = None, y: Optional[
 def latent_store(proj: torch.Tensor, q_offset: int, q_weight: Optional[torch.Tensor], q_latent: Optional[torch.Tensor],
                  c_offset: int, c_weight: torch.Tensor, rot_offset: int, freq: Optional[torch.Tensor], amplitude: float,
                  eps: float, positions: torch.Tensor, row_req: torch.Tensor, block_tables: torch.Tensor, cache: torch.Tensor,
-                 page_size: int, write_cache: bool = True) -> None:
+                 page_size: int, write_cache: bool = True, interleaved: bool = True) -> None:
     """From the 32-bit projections ``proj`` [T, ld]: the query latent (columns from q_offset, len(q_weight) wide) is
     brought to unit RMS, weighted and written to ``q_latent`` [T, q_rank]; the key/value latent (from c_offset,
     len(c_weight) wide) likewise into the first columns of the token's page row of ``cache`` [pages, 1, page_size,
-    rank + rot]; the 2 * len(freq) columns from rot_offset are rotated pair by pair (2i, 2i+1) by position * freq[i],
-    cos and sin times ``amplitude``, and written behind it."""
+    rank + rot]; the 2 * len(freq) columns from rot_offset are rotated pair by pair ((2i, 2i+1), or (i, i + len(freq)) when
+    not ``interleaved``) by position * freq[i], cos and sin times ``amplitude``, and written behind it."""
     T, ld = proj.shape
     rank = c_weight.numel()
     rot = 0 if freq is None else 2 * freq.numel()
@@ -464,7 +502,7 @@ def latent_store(proj: torch.Tensor, q_offset: int, q_weight: Optional[torch.Ten
         _dev(proj, "proj", torch.float32), ld, int(q_offset), 0 if q_weight is None else q_weight.numel(),
         _opt(q_weight, "q_weight", torch.float32), 0 if q_latent is None else _dev(q_latent, "q_latent"), int(c_offset), rank,
         _dev(c_weight, "c_weight", torch.float32), int(rot_offset), rot, _opt(freq, "freq", torch.float32), float(amplitude),
-        float(eps), _dev(positions, "positions", torch.int32), _dev(row_req, "row_req", torch.int32),
+        int(interleaved), float(eps), _dev(positions, "positions", torch.int32), _dev(row_req, "row_req", torch.int32),
         _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1], _dev(cache, "cache"), dtype_code(cache.dtype), T,
         page_size, int(write_cache), _stream()), "latent_store")
 
@@ -514,12 +552,13 @@ def attention_rows(q: torch.Tensor, k_cache: torch.Tensor, v_cache: Optional[tor
                    window: Optional[int] = None, chunk: Optional[int] = None, slopes: Optional[torch.Tensor] = None,
                    sinks: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
                    tiles: Optional[torch.Tensor] = None, splits: int = 1, workspace: Optional[torch.Tensor] = None,
-                   softcap: Optional[float] = None) -> None:
+                   softcap: Optional[float] = None, gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
     """Attention of every row of ``q`` [T, H*hd] (32-bit or bfloat16) over its request's pages, 32-bit arithmetic.
     ``v_cache`` None: the values are the first ``value_dim`` columns of the key rows. ``window``: the last w positions;
     ``chunk``: only keys of the query's own block of c positions; ``slopes`` [H]: slope_h * distance is taken off a
     score; ``sinks`` [H]: exp(sinks_h) more in the softmax's denominator; ``softcap`` c: the scaled score s becomes
-    c tanh(s / c). ``out`` [T, H*vd], 32-bit or bfloat16.
+    c tanh(s / c); ``gate`` [T, ld] 32-bit: output column c is multiplied by sigmoid(gate[t, gate_offset + c]).
+    ``out`` [T, H*vd], 32-bit or bfloat16.
     (See attention_rows_tensor_cores for the form that rounds queries and softmax weights to bfloat16.)
     Tensor-core form only (attention_rows_tile_tokens() > 0): ``rows`` [n] lists the step rows to work on, a tile each;
     ``tiles`` [m, 3] = (first row, tokens (at most attention_rows_tile_tokens()), request) lists tiles of consecutive
@@ -540,13 +579,15 @@ def attention_rows(q: torch.Tensor, k_cache: torch.Tensor, v_cache: Optional[tor
     for t, name in ((slopes, "slopes"), (sinks, "sinks")):
         if t is not None and t.numel() != num_heads:
             raise KernelError(f"attention_rows: {name} must have one value per head")
+    if gate is not None and (gate.dim() != 2 or gate.shape[0] != T or gate_offset < 0 or gate_offset + num_heads * value_dim > gate.shape[1]):
+        raise KernelError("attention_rows: the gate must be [T, ld] with the output's columns inside a row")
     check(lib().gi_attention_rows(
         _dev(q, "q"), dtype_code(q.dtype), q.shape[1], _dev(k_cache, "k_cache"), 0 if v_cache is None else _dev(v_cache, "v_cache"),
         dtype_code(k_cache.dtype), _dev(out, "out"), dtype_code(out.dtype), out.shape[1], _dev(row_req, "row_req", torch.int32),
         _dev(positions, "positions", torch.int32), _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1], T,
         num_heads, num_kv_heads, head_dim, value_dim, head_dim if v_cache is None else value_dim, int(v_cache is None), page_size,
         float(scale), float(softcap or 0.0), int(window or 0), int(chunk or 0), _opt(slopes, "slopes", torch.float32), _opt(sinks, "sinks", torch.float32),
-        _opt(lst, "rows or tiles", torch.int32), kind, n_list, int(splits), _opt(workspace, "workspace", torch.float32),
+        _opt(gate, "gate", torch.float32), 0 if gate is None else gate.shape[1], int(gate_offset), _opt(lst, "rows or tiles", torch.int32), kind, n_list, int(splits), _opt(workspace, "workspace", torch.float32),
         0 if workspace is None else workspace.numel(), _stream()), "attention_rows")
     if splits > 1:
         count_launches(1)
@@ -555,13 +596,14 @@ def attention_rows(q: torch.Tensor, k_cache: torch.Tensor, v_cache: Optional[tor
 def attention_rows_of_step(ctx, q: torch.Tensor, k_cache: torch.Tensor, v_cache: Optional[torch.Tensor], out: torch.Tensor,
                            tables: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, scale: float,
                            window: Optional[int], chunk: Optional[int], slopes: Optional[torch.Tensor],
-                           sinks: Optional[torch.Tensor], softcap: Optional[float] = None, tiles_on=None, singles_on=None) -> None:
+                           sinks: Optional[torch.Tensor], softcap: Optional[float] = None, tiles_on=None, singles_on=None,
+                           gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
     """``attention_rows`` for all rows of a step. Over a bfloat16 cache with sizes that the tensor-core form serves, the
     step's single tokens and the tiles of its prompt portions (``ctx.attention_work``) run as two launches, each with its
     keys cut into ranges when it has few tiles; otherwise one launch works row by row. ``tiles_on`` = (tokens per tile,
     fn(work)): the tiles of prompt portions go to ``fn`` instead, another kernel that serves this form of attention;
     ``singles_on`` = fn(rows, longest context): likewise the rows of requests that bring a single token."""
-    common = dict(window=window, chunk=chunk, slopes=slopes, sinks=sinks, softcap=softcap)
+    common = dict(window=window, chunk=chunk, slopes=slopes, sinks=sinks, softcap=softcap, gate=gate, gate_offset=gate_offset)
     per_tile = attention_rows_tile_tokens(num_heads, num_kv_heads, head_dim, value_dim, v_cache is None) \
         if k_cache.dtype is torch.bfloat16 else 0
     if per_tile == 0 or not hasattr(ctx, "attention_work"):
@@ -603,15 +645,18 @@ def attention_rows_launch_key(ctx, num_heads: int, num_kv_heads: int, head_dim: 
 
 def head_product(a: torch.Tensor, a_offset: int, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_offset: int,
                  out_head_stride: int, tail: int = 0, freq: Optional[torch.Tensor] = None, amplitude: float = 1.0,
-                 positions: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_offset: int = 0) -> None:
+                 positions: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
+                 interleaved: bool = True, gate_per_head: bool = False) -> None:
     """out[t, out_offset + h * out_head_stride + n] = sum_k w[h, n, k] * a[t, a_offset + h * a_head_stride + k] for
     every head h of ``w`` [H, N, K]: a matrix per head, applied to that head's slice of a row. ``tail`` > 0: the tail
-    columns behind a head's K inputs are rotated pair by pair by positions[t] * freq[i] (cos and sin times
-    ``amplitude``) and written behind the head's N outputs. ``gate`` [T, ld] 32-bit: output n of head h is multiplied by
-    sigmoid(gate[t, gate_offset + h * N + n]) (an element-wise output gate laid out head by head)."""
+    columns behind a head's K inputs are rotated pair by pair ((2i, 2i+1), or (i, i + tail / 2) when not ``interleaved``)
+    by positions[t] * freq[i] (cos and sin times ``amplitude``) and written behind the head's N outputs. ``gate`` [T, ld] 32-bit: output n of head h is multiplied by
+    sigmoid(gate[t, gate_offset + h * N + n]) (an element-wise output gate laid out head by head), with ``gate_per_head``
+    by sigmoid(gate[t, gate_offset + h])."""
     T = a.shape[0]
     H, N, K = w.shape
-    if gate is not None and (gate.dim() != 2 or gate.shape[0] != T or gate_offset < 0 or gate_offset + H * N > gate.shape[1]):
+    if gate is not None and (gate.dim() != 2 or gate.shape[0] != T or gate_offset < 0 or
+                             gate_offset + H * (1 if gate_per_head else N) > gate.shape[1]):
         raise KernelError("head_product: the gate's columns lie outside its rows")
     if a.dim() != 2 or out.dim() != 2 or out.shape[0] != T:
         raise KernelError("head_product: a and out must be matrices with one row per token")
@@ -622,8 +667,8 @@ def head_product(a: torch.Tensor, a_offset: int, a_head_stride: int, w: torch.Te
     check(lib().gi_head_product(
         _dev(a, "a"), dtype_code(a.dtype), a.shape[1], int(a_offset), int(a_head_stride), _dev(w, "w"), dtype_code(w.dtype), N * K,
         _dev(out, "out"), dtype_code(out.dtype), out.shape[1], int(out_offset), int(out_head_stride), T, H, N, K, int(tail),
-        _opt(freq, "freq", torch.float32), float(amplitude), 0 if positions is None else _dev(positions, "positions", torch.int32),
-        _opt(gate, "gate", torch.float32), 0 if gate is None else gate.shape[1], int(gate_offset), _stream()), "head_product")
+        _opt(freq, "freq", torch.float32), float(amplitude), int(interleaved), 0 if positions is None else _dev(positions, "positions", torch.int32),
+        _opt(gate, "gate", torch.float32), 0 if gate is None else gate.shape[1], int(gate_offset), int(gate_per_head), _stream()), "head_product")
 
 
 def grouped_tile_rows() -> int:
@@ -644,14 +689,16 @@ def route_tiles(n_tokens: int, top: int, experts: int, tile_rows: Optional[int] 
 def route(x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tensor], top: int, ids: torch.Tensor,
           weights: torch.Tensor, sorted_rows: torch.Tensor, tile_group: torch.Tensor, n_tiles: torch.Tensor,
           tile_rows: Optional[int] = None, pair_row: Optional[torch.Tensor] = None, scores: str = "sigmoid",
-          renormalise: bool = False, factor: float = 1.0) -> None:
+          renormalise: bool = False, factor: float = 1.0, gate_w: Optional[torch.Tensor] = None, gate_out: Optional[torch.Tensor] = None) -> None:
     """Per row of ``x`` [T, D]: s = sigmoid(w x) with ``w`` [E, D] 32-bit (``scores`` "softmax": s = softmax(w x) over all
     experts); the ``top`` experts with the largest s + correction go to ``ids`` [T, top] and their s to ``weights`` [T, top]
     (``renormalise``: divided by the chosen ones' sum + 1e-20), times ``factor``. The pairs (token, choice) are then
     bucketed by expert into tiles of ``tile_rows`` rows (grouped_tile_rows() by default): ``sorted_rows`` (pair index
     or -1), ``tile_group`` (a tile's expert), ``n_tiles`` [1], and optionally ``pair_row`` [T * top], the row each pair
-    landed in. Two launches."""
+    landed in. ``gate_w`` [D] 32-bit with ``gate_out`` [T]: also gate_out = sigmoid(gate_w x). Two launches."""
     T, D = x.shape
+    if (gate_w is None) != (gate_out is None) or (gate_w is not None and (gate_w.numel() != D or gate_out.numel() != T)):
+        raise KernelError("route: a gate needs a row of D weights and a place for T values")
     E = w.shape[0]
     max_tiles = tile_group.numel()
     tm = tile_rows or grouped_tile_rows()
@@ -664,7 +711,8 @@ def route(x: torch.Tensor, w: torch.Tensor, correction: Optional[torch.Tensor], 
     check(lib().gi_route(_dev(x, "x"), dtype_code(x.dtype), T, D, _dev(w, "w", torch.float32), _opt(correction, "correction", torch.float32),
                          E, int(top), int(scores == "softmax"), int(bool(renormalise)), float(factor), _dev(ids, "ids", torch.int32), _dev(weights, "weights", torch.float32),
                          _dev(sorted_rows, "sorted_rows", torch.int32), _dev(tile_group, "tile_group", torch.int32),
-                         _dev(n_tiles, "n_tiles", torch.int32), max_tiles, tm, _opt(pair_row, "pair_row", torch.int32), _stream()), "route")
+                         _dev(n_tiles, "n_tiles", torch.int32), max_tiles, tm, _opt(pair_row, "pair_row", torch.int32),
+                         _opt(gate_w, "gate_w", torch.float32), _opt(gate_out, "gate_out", torch.float32), _stream()), "route")
     count_launches(1)
 
 
@@ -689,12 +737,15 @@ def route_table(tokens: torch.Tensor, feedback: Optional[torch.Tensor], table: t
     count_launches(1)
 
 
-def gather_rows(x: torch.Tensor, a_div: int, sorted_rows: torch.Tensor, n_tiles: torch.Tensor, tile_rows: int, out: torch.Tensor) -> None:
-    """out[r] = x[sorted_rows[r] // a_div] for the rows of the first n_tiles tiles (zeros where sorted_rows is -1)."""
+def gather_rows(x: torch.Tensor, a_div: int, sorted_rows: torch.Tensor, n_tiles: torch.Tensor, tile_rows: int, out: torch.Tensor,
+                scales: Optional[torch.Tensor] = None) -> None:
+    """out[r] = x[sorted_rows[r] // a_div] for the rows of the first n_tiles tiles (zeros where sorted_rows is -1); ``scales``
+    32-bit, one per pair: times scales[sorted_rows[r]]."""
     if out.shape[1] != x.shape[1] or out.dtype != x.dtype or sorted_rows.numel() < out.shape[0]:
         raise KernelError("gather_rows: shapes do not agree")
     check(lib().gi_gather_rows(_dev(x, "x"), dtype_code(x.dtype), x.shape[1], int(a_div), _dev(sorted_rows, "sorted_rows", torch.int32),
-                               _dev(n_tiles, "n_tiles", torch.int32), int(tile_rows), out.shape[0], _dev(out, "out"), _stream()), "gather_rows")
+                               _dev(n_tiles, "n_tiles", torch.int32), int(tile_rows), out.shape[0], _opt(scales, "scales", torch.float32),
+                               _dev(out, "out"), _stream()), "gather_rows")
 
 
 def expert_product_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tile_group: torch.Tensor, n_tiles: torch.Tensor,
@@ -726,10 +777,11 @@ def expert_product_tc_supported(N: int, K: int, gated: bool) -> bool:
 
 def expert_product(a: torch.Tensor, a_div: int, w: torch.Tensor, out: torch.Tensor, sorted_rows: torch.Tensor,
                    tile_group: torch.Tensor, n_tiles: torch.Tensor, gated: Optional[str] = None, limit: float = 0.0,
-                   act: Optional[str] = None) -> None:
+                   act: Optional[str] = None, scales: Optional[torch.Tensor] = None) -> None:
     """out[pair] = W[expert of pair] a[pair // a_div] for the pairs that ``route`` bucketed, ``w`` [E, N, K] (gated:
     [E, 2N, K], gate rows first, and out = act(gate) * up with ``gated`` one of ACTIVATIONS). ``act``: one of
-    PLAIN_ACTIVATIONS on the output of an ungated product."""
+    PLAIN_ACTIVATIONS on the output of an ungated product. ``scales`` 32-bit, one per pair: the product's values (gate and
+    up alike) are multiplied by it before the activation, as if the pair's input row had been."""
     if act is not None and (gated is not None or act not in PLAIN_ACTIVATIONS):
         raise KernelError(f"expert_product: unknown activation '{act}' (or one beside a gated one)")
     E, rows, K = w.shape
@@ -740,22 +792,27 @@ def expert_product(a: torch.Tensor, a_div: int, w: torch.Tensor, out: torch.Tens
         raise KernelError(f"expert_product: unknown activation '{gated}'")
     check(lib().gi_expert_product(_dev(a, "a"), dtype_code(a.dtype), K, int(a_div), _dev(w, "w"), dtype_code(w.dtype), rows * K, K,
                                   N * K if gated else 0, int(gated is not None),
-                                  ACTIVATIONS[gated] if gated else PLAIN_ACTIVATIONS[act or "none"], float(limit), _dev(out, "out"),
-                                  dtype_code(out.dtype), N, N, K, _dev(tile_group, "tile_group", torch.int32),
+                                  ACTIVATIONS[gated] if gated else PLAIN_ACTIVATIONS[act or "none"], float(limit),
+                                  _opt(scales, "scales", torch.float32), _dev(out, "out"), dtype_code(out.dtype), N, N, K, _dev(tile_group, "tile_group", torch.int32),
                                   _dev(sorted_rows, "sorted_rows", torch.int32), _dev(n_tiles, "n_tiles", torch.int32),
                                   tile_group.numel(), _stream()), "expert_product")
 
 
-def route_combine(part: torch.Tensor, weights: torch.Tensor, y: torch.Tensor, pair_row: Optional[torch.Tensor] = None) -> None:
+def route_combine(part: torch.Tensor, weights: Optional[torch.Tensor], y: torch.Tensor, pair_row: Optional[torch.Tensor] = None,
+                  top: Optional[int] = None, more: Optional[torch.Tensor] = None, more_gate: Optional[torch.Tensor] = None) -> None:
     """y[t] += sum_k weights[t, k] * part[row of pair t * top + k], in the order of k; all 32-bit. The row of a pair is
-    the pair itself, or ``pair_row[pair]`` when given."""
+    the pair itself, or ``pair_row[pair]`` when given. ``weights`` None (then ``top`` says how many): weights of 1.
+    ``more`` [T, D] with ``more_gate`` [T]: plus more_gate[t] * more[t]."""
     T, D = y.shape
-    top = weights.shape[1]
-    if part.dim() != 2 or part.shape[1] != D or weights.shape[0] != T or (pair_row is None and part.shape[0] != T * top) or \
+    top = int(top) if weights is None else weights.shape[1]
+    if (more is None) != (more_gate is None) or (more is not None and (more.shape != y.shape or more_gate.numel() != T)):
+        raise KernelError("route_combine: a gated part must be [T, D] with a gate per row")
+    if part.dim() != 2 or part.shape[1] != D or (weights is not None and weights.shape[0] != T) or (pair_row is None and part.shape[0] != T * top) or \
             (pair_row is not None and pair_row.numel() < T * top):
         raise KernelError("route_combine: shapes do not agree")
-    check(lib().gi_route_combine(_dev(part, "part", torch.float32), _dev(weights, "weights", torch.float32),
-                                 _opt(pair_row, "pair_row", torch.int32), _dev(y, "y", torch.float32), T, D, top, _stream()), "route_combine")
+    check(lib().gi_route_combine(_dev(part, "part", torch.float32), _opt(weights, "weights", torch.float32),
+                                 _opt(pair_row, "pair_row", torch.int32), _opt(more, "more", torch.float32),
+                                 _opt(more_gate, "more_gate", torch.float32), _dev(y, "y", torch.float32), T, D, top, _stream()), "route_combine")
 
 
 def causal_conv(proj: torch.Tensor, offset: int, weight: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor,
@@ -926,13 +983,13 @@ def attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                       row_req: torch.Tensor, positions: torch.Tensor, block_tables: torch.Tensor,
                       num_heads: int, num_kv_heads: int, head_dim: int, page_size: int, scale: float,
                       window: Optional[int] = None, sink: bool = False, gate: Optional[torch.Tensor] = None,
-                      gate_offset: int = 0, out_scale: float = 1.0) -> None:
+                      gate_offset: int = 0, out_scale: float = 1.0, gate_dims: int = 0) -> None:
     """Causal attention of every row of ``q`` [T, H*hd] over its request's pages. ``sink``: one more in the
-    softmax's denominator; ``gate`` [T, ld] 32-bit: head h's output times sigmoid(gate[t, gate_offset + h]);
-    ``out_scale``: a constant factor on the output."""
+    softmax's denominator; ``gate`` [T, ld] 32-bit: head h's output times sigmoid(gate[t, gate_offset + h]), or with
+    ``gate_dims`` = hd value d of it times sigmoid(gate[t, gate_offset + h * hd + d]); ``out_scale``: a constant factor on
+    the output."""
     T = q.shape[0]
-    if gate is not None and (gate.dim() != 2 or gate.shape[0] != T or gate_offset < 0 or gate_offset + num_heads > gate.shape[1]):
-        raise KernelError("attention: the gate must be [T, ld] with the heads' columns inside a row")
+    epilogue = _epilogue(sink, gate, gate_offset, out_scale, num_heads, gate_dims, head_dim, T)
     if q.shape != (T, num_heads * head_dim) or out.shape != q.shape or out.dtype != q.dtype:
         raise KernelError("attention: q and out must be [T, H*hd] of one dtype")
     if k_cache.dtype != q.dtype or v_cache.dtype != q.dtype:
@@ -943,16 +1000,19 @@ def attention_generic(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         _dev(q, "q"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), _dev(out, "out"), dtype_code(q.dtype),
         _dev(row_req, "row_req", torch.int32), _dev(positions, "positions", torch.int32),
         _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1], T, num_heads, num_kv_heads,
-        head_dim, page_size, float(scale), int(window or 0), int(bool(sink)), _opt(gate, "gate", torch.float32),
-        0 if gate is None else gate.shape[1], int(gate_offset), float(out_scale), _stream()), "attention")
+        head_dim, page_size, float(scale), int(window or 0), *epilogue, _stream()), "attention")
 
 
-def _epilogue(sink: bool, gate: Optional[torch.Tensor], gate_offset: int, out_scale: float, num_heads: int):
+def _epilogue(sink: bool, gate: Optional[torch.Tensor], gate_offset: int, out_scale: float, num_heads: int, gate_dims: int,
+              head_dim: int, rows: int):
     """The arguments every attention entry point takes for what follows the softmax: a sink in the denominator,
-    a sigmoid gate per head read from a 32-bit [T, ld] tensor, a constant factor."""
-    if gate is not None and (gate.dim() != 2 or gate_offset < 0 or gate_offset + num_heads > gate.shape[1]):
+    a sigmoid gate per head (or per value: ``gate_dims`` = head_dim) read from a 32-bit [T, ld] tensor, a constant factor."""
+    if gate_dims not in (0, head_dim) or (gate_dims and gate is None):
+        raise KernelError("attention: a gate has one value per head or one per value of a head")
+    if gate is not None and (gate.dim() != 2 or gate.shape[0] != rows or gate_offset < 0 or
+                             gate_offset + num_heads * (gate_dims or 1) > gate.shape[1]):
         raise KernelError("attention: the gate must be [T, ld] with the heads' columns inside a row")
-    return (int(bool(sink)), _opt(gate, "gate", torch.float32), 0 if gate is None else gate.shape[1], int(gate_offset),
+    return (int(bool(sink)), _opt(gate, "gate", torch.float32), 0 if gate is None else gate.shape[1], int(gate_offset), int(gate_dims),
             float(out_scale))
 
 
@@ -986,10 +1046,10 @@ def attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      num_heads: int, num_kv_heads: int, head_dim: int, page_size: int, scale: float,
                      window: Optional[int], part_o: torch.Tensor, part_ml: torch.Tensor, max_chunks: int,
                      n_chunks: int, sink: bool = False, gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
-                     out_scale: float = 1.0, softcap: Optional[float] = None) -> None:
+                     out_scale: float = 1.0, softcap: Optional[float] = None, gate_dims: int = 0) -> None:
     """Attention of single decoded tokens (bfloat16): ``rows`` lists their step rows; the context is
     split into fixed chunks whose partial results go through ``part_o`` / ``part_ml``. ``sink``, ``gate``,
-    ``gate_offset``, ``out_scale``: as in ``attention_generic``. ``softcap`` c (pages that ``attention_tma_pages`` accepts
+    ``gate_offset``, ``gate_dims``, ``out_scale``: as in ``attention_generic``. ``softcap`` c (pages that ``attention_tma_pages`` accepts
     only): the scaled score s becomes c tanh(s / c)."""
     n = rows.numel()
     if part_o.numel() < n * num_heads * max_chunks * head_dim or part_ml.numel() < n * num_heads * max_chunks * 2:
@@ -1004,7 +1064,7 @@ def attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         _dev(positions, "positions", torch.int32), _dev(block_tables, "block_tables", torch.int32),
         block_tables.shape[1], num_heads, num_kv_heads, head_dim, page_size, float(scale), int(window or 0),
         _dev(part_o, "part_o", torch.float32), _dev(part_ml, "part_ml", torch.float32), max_chunks, n_chunks,
-        k_cache.shape[0], _tc_state(q.device).status.data_ptr(), *_epilogue(sink, gate, gate_offset, out_scale, num_heads),
+        k_cache.shape[0], _tc_state(q.device).status.data_ptr(), *_epilogue(sink, gate, gate_offset, out_scale, num_heads, gate_dims, head_dim, q.shape[0]),
         float(softcap or 0.0), _stream()), "attention_decode")
     tma = page_size % 8 == 0 and (32 % page_size == 0 or page_size % 32 == 0)
     if n_chunks > 1 or not tma:
@@ -1015,7 +1075,7 @@ def attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                       work: torch.Tensor, positions: torch.Tensor, block_tables: torch.Tensor, num_heads: int,
                       num_kv_heads: int, head_dim: int, page_size: int, scale: float, window: Optional[int],
                       sink: bool = False, gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
-                      out_scale: float = 1.0) -> None:
+                      out_scale: float = 1.0, gate_dims: int = 0) -> None:
     """Attention of prompt portions (bfloat16): ``work`` [n, 3] = (first step row of a tile, tokens
     in it (at most attention_prefill_rows() // group size), request index)."""
     if work.dim() != 2 or work.shape[1] != 3:
@@ -1029,7 +1089,7 @@ def attention_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         _dev(out, "out", torch.bfloat16), _dev(work, "work", torch.int32), work.shape[0],
         _dev(positions, "positions", torch.int32), _dev(block_tables, "block_tables", torch.int32),
         block_tables.shape[1], num_heads, num_kv_heads, head_dim, page_size, float(scale), int(window or 0),
-        k_cache.shape[0], _tc_state(q.device).status.data_ptr(), *_epilogue(sink, gate, gate_offset, out_scale, num_heads),
+        k_cache.shape[0], _tc_state(q.device).status.data_ptr(), *_epilogue(sink, gate, gate_offset, out_scale, num_heads, gate_dims, head_dim, q.shape[0]),
         _stream()), "attention_prefill")
 
 
@@ -1042,7 +1102,7 @@ def attention_prefill_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
                          work: torch.Tensor, positions: torch.Tensor, block_tables: torch.Tensor, num_heads: int,
                          num_kv_heads: int, head_dim: int, page_size: int, scale: float, window: Optional[int],
                          sink: bool = False, gate: Optional[torch.Tensor] = None, gate_offset: int = 0,
-                         out_scale: float = 1.0, softcap: Optional[float] = None) -> None:
+                         out_scale: float = 1.0, softcap: Optional[float] = None, gate_dims: int = 0) -> None:
     """Attention of prompt portions on the tcgen05 tensor cores: ``work`` [n, 3] = (first step row of
     a tile, tokens in it (at most 128 // group size), request index). ``softcap`` c: the scaled score s becomes c tanh(s / c)."""
     if work.dim() != 2 or work.shape[1] != 3:
@@ -1056,7 +1116,7 @@ def attention_prefill_tc(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.
         _dev(out, "out", torch.bfloat16), _dev(work, "work", torch.int32), work.shape[0],
         _dev(positions, "positions", torch.int32), _dev(block_tables, "block_tables", torch.int32),
         block_tables.shape[1], num_heads, num_kv_heads, head_dim, page_size, float(scale), int(window or 0),
-        k_cache.shape[0], _tc_state(q.device).status.data_ptr(), *_epilogue(sink, gate, gate_offset, out_scale, num_heads),
+        k_cache.shape[0], _tc_state(q.device).status.data_ptr(), *_epilogue(sink, gate, gate_offset, out_scale, num_heads, gate_dims, head_dim, q.shape[0]),
         float(softcap or 0.0), _stream()), "attention_prefill_tc")
 
 

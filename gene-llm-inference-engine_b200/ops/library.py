@@ -26,32 +26,36 @@ _SIGNATURES = {
                       c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "gi_copy_pages": [c_void_p, c_longlong, c_int, c_longlong, c_void_p, c_void_p, c_int, c_void_p],
     "gi_attention_generic": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                             c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_float,
+                             c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_int, c_float,
                              c_void_p],
     "gi_scale_cast": [c_void_p, c_void_p, c_void_p, c_int, c_float, c_longlong, c_void_p],
     "gi_residual_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p],
     "gi_gated_act": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p],
-    "gi_norm_rope_store": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int,
+    "gi_norm_rope_store": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int,
                            c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                            c_int, c_int, c_int, c_int, c_int, c_void_p],
     "gi_add_normed": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
     "gi_latent_store": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p,
-                        c_float, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+                        c_float, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "gi_attention_rows": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p,
                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_int,
-                          c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p],
+                          c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_longlong, c_void_p],
     "gi_attention_rows_tile_tokens": [c_int, c_int, c_int, c_int, c_int],
     "gi_attention_rows_supported": [c_int, c_int],
     "gi_attention_rows_set_mma": [c_int],
     "gi_attention_rows_set_pairs": [c_int],
     "gi_head_product": [c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong,
-                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_longlong, c_int, c_void_p],
+                        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_int, c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p],
     "gi_expert_product": [c_void_p, c_int, c_longlong, c_int, c_void_p, c_int, c_longlong, c_int, c_longlong, c_int, c_int, c_float,
-                          c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                          c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     "gi_route": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
-                 c_void_p, c_int, c_int, c_void_p, c_void_p],
-    "gi_gather_rows": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
-    "gi_route_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+                 c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+    "gi_gather_rows": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    "gi_add_stream": [c_void_p, c_void_p, c_longlong, c_void_p],
+    "gi_dynamic_tanh": [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "gi_add_dynamic_tanh": [c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int,
+                            c_int, c_int, c_int, c_void_p],
+    "gi_route_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "gi_gemm_tc_grouped": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p],
     "gi_route_table": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                        c_int, c_int, c_void_p, c_void_p],
@@ -99,9 +103,9 @@ _SIGNATURES = {
     "gi_gemm_tc_status": [c_void_p, c_void_p, c_void_p],
     "gi_attention_decode": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                             c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_longlong,
-                            c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_float, c_void_p],
+                            c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_float, c_void_p],
     "gi_attention_prefill": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-                             c_int, c_int, c_int, c_float, c_int, c_longlong, c_void_p, c_int, c_void_p, c_int, c_int, c_float,
+                             c_int, c_int, c_int, c_float, c_int, c_longlong, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float,
                              c_void_p],
     "gi_attention_prefill_rows": [c_int, c_int],
     "gi_gemm_tc_set_cluster": [c_int],
@@ -112,7 +116,7 @@ _SIGNATURES = {
     "gi_attention_set_stream_kv": [c_int],
     "gi_gemm_tc_cluster_capacity": [c_int, c_int, c_int],
     "gi_attention_prefill_tc": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-                                c_int, c_int, c_int, c_float, c_int, c_longlong, c_void_p, c_int, c_void_p, c_int, c_int,
+                                c_int, c_int, c_int, c_float, c_int, c_longlong, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
                                 c_float, c_float, c_void_p],
     "gi_attention_prefill_tc_supported": [c_int, c_int, c_int, c_int],
     "gi_attention_fast_supported": [c_int, c_int, c_int],

@@ -44,6 +44,10 @@ class AttentionMixer:
     nothing before the first token; one tap is a factor per channel); the request's last n-1 projected rows are state, kept
     in its state slot from ``state_offset`` on.
 
+    ``bias``: q, k and v have biases, added in 32-bit to the projection before the norm and the rotation (``b_qkv`` [(H + Hkv) hd +
+    Hkv vd]). ``output_gate``: ``w_qkv`` ends with H vd more rows, and every value of the heads' outputs is multiplied by the
+    sigmoid of its row's product with the input (in the attention kernels' last step).
+
     ``maps`` = 2 (with ``map_weight`` and ``map_factor``): every head has two score maps over the same values. ``num_heads`` and
     ``num_kv_heads`` count heads, ``head_dim`` is the width of one map; a head's queries and keys are [map 1, map 2] in
     ``w_qkv`` (2 H hd query rows, 2 Hkv hd key rows), each map brought to unit RMS and weighted on its own (``qk_norm_eps``,
@@ -104,9 +108,14 @@ class AttentionMixer:
                 not kernels.attention_fast_supported(self.head_dim, self.num_heads, self.num_kv_heads)
         self.sink = bool(params.get("sink", False))
         self.head_gate = bool(params.get("head_gate", False))
+        self.output_gate = bool(params.get("output_gate", False))
+        if self.output_gate and (self.head_gate or params.get("conv_taps") or self.maps == 2):
+            raise ValueError("attention: an output gate cannot be combined with a head gate, a convolution or two score maps")
+        if params.get("bias") and (self.values_are_keys or params.get("conv_taps") or self.maps == 2):
+            raise ValueError("attention: biases cannot be combined with values taken from the keys, a convolution or two score maps")
         self.out_scale = float(params.get("out_scale", 1.0))
         on_device = getattr(self.position, "freq", None) is not None
-        self.extended = (self.values_are_keys or self.qk_norm_eps is not None or self.sink or self.head_gate
+        self.extended = (self.output_gate or bool(params.get("bias")) or self.values_are_keys or self.qk_norm_eps is not None or self.sink or self.head_gate
                          or self.out_scale != 1.0 or on_device or self.row_form or self.conv_taps is not None)
         if self.row_form:
             if self.head_gate or self.out_scale != 1.0 or self.values_are_keys:
@@ -148,13 +157,19 @@ class AttentionMixer:
             out_columns = self.map_heads * self.map_value_dim
         else:
             qkv_rows = (self.num_heads + self.num_kv_heads) * self.head_dim + \
-                (0 if self.values_are_keys else self.num_kv_heads * self.value_dim) + (self.num_heads if self.head_gate else 0)
+                (0 if self.values_are_keys else self.num_kv_heads * self.value_dim) + (self.num_heads if self.head_gate else 0) + \
+                (self.num_heads * self.value_dim if self.output_gate else 0)
             out_columns = self.num_heads * self.value_dim
         if tuple(weights["w_qkv"].shape) != (qkv_rows, self.hidden_size):
             raise ValueError(f"attention: w_qkv has shape {tuple(weights['w_qkv'].shape)}, expected "
                              f"({qkv_rows}, {self.hidden_size})")
         if tuple(weights["w_o"].shape) != (self.hidden_size, out_columns):
             raise ValueError(f"attention: w_o has shape {tuple(weights['w_o'].shape)}")
+        self.bias = None
+        if params.get("bias"):          # zeros behind: a gate's columns have none
+            n = (self.num_heads + self.num_kv_heads) * self.head_dim + self.num_kv_heads * self.value_dim
+            self.bias = torch.zeros(qkv_rows, dtype=torch.float32, device=build.device)
+            self.bias[:n] = _vector_of(weights, "b_qkv", n, build)
         self.conv = None
         if self.conv_taps is not None:
             if self.head_gate or self.values_are_keys:
@@ -271,7 +286,7 @@ class AttentionMixer:
 
     def _attend(self, ctx, q, k_cache, v_cache, att, tables, **epilogue) -> None:
         """Attention of the step's rows: single decoded tokens split their context over many CTAs, portions of
-        prompts run tile by tile (tensor cores); else the general kernel. ``epilogue``: sink, gate, gate_offset, out_scale."""
+        prompts run tile by tile (tensor cores); else the general kernel. ``epilogue``: sink, gate, gate_offset, gate_dims, out_scale."""
         H, Hkv, hd = self.num_heads, self.num_kv_heads, self.head_dim
         if not self._fast_now(ctx):
             kernels.attention_generic(q, k_cache, v_cache, att, ctx.row_req, ctx.positions, tables, H, Hkv, hd,
@@ -342,18 +357,21 @@ class AttentionMixer:
             return
         k_off = H * hd
         v_off = k_off if self.values_are_keys else k_off + Hkv * hd
-        gate_off = v_off + Hkv * hd
+        gate_off = v_off + Hkv * self.value_dim
         kernels.norm_rope_store(proj, 0, k_off, v_off, self.q_norm, self.k_norm, self.qk_norm_eps or 0.0,
                                 getattr(self.position, "freq", None), self.position.interleaved, ctx.positions,
                                 ctx.row_req, tables, q, k_cache, v_cache, H, Hkv, hd, ctx.page_size,
-                                write_kv=run.writes_cache, value_dim=self.value_dim, wide_norm=self.wide_norm)
+                                write_kv=run.writes_cache, value_dim=self.value_dim, wide_norm=self.wide_norm, bias=self.bias)
+        # (a gate per head, or one per value laid out as the heads' outputs)
+        gate = {"gate": proj if self.head_gate or self.output_gate else None, "gate_offset": gate_off}
+        gate_dims = self.value_dim if self.output_gate else 0
         if self.row_form:
             att = ctx.scratch("att", (T, H * self.value_dim), self.dtype)
             tiles_on = None
             if self._cap_tiles_on_tcgen05(ctx):
                 tiles_on = (128 // (H // Hkv), lambda work: kernels.attention_prefill_tc(
                     q, k_cache, v_cache, att, work, ctx.positions, tables, H, Hkv, hd, ctx.page_size, self.scale, self.window,
-                    softcap=self.softcap))
+                    softcap=self.softcap, gate_dims=gate_dims, **gate))
             singles_on = None
             if self._cap_singles_on_decode(ctx):
                 def singles_on(rows, longest):
@@ -362,15 +380,15 @@ class AttentionMixer:
                     part_ml = ctx.scratch("att_part_ml", (n, H * self.max_chunks * 2), torch.float32, capacity=ctx.max_requests)
                     kernels.attention_decode(q, k_cache, v_cache, att, rows, ctx.row_req, ctx.positions, tables, H, Hkv, hd,
                                              ctx.page_size, self.scale, self.window, part_o, part_ml, self.max_chunks,
-                                             (longest + self.chunk_keys - 1) // self.chunk_keys, softcap=self.softcap)
+                                             (longest + self.chunk_keys - 1) // self.chunk_keys, softcap=self.softcap,
+                                             gate_dims=gate_dims, **gate)
             kernels.attention_rows_of_step(ctx, q, k_cache, v_cache, att, tables, H, Hkv, hd, self.value_dim, self.scale,
                                            self.window, self.chunk, self.slopes, self.sink_weight, softcap=self.softcap,
-                                           tiles_on=tiles_on, singles_on=singles_on)
+                                           tiles_on=tiles_on, singles_on=singles_on, **gate)
             self.w_o.forward(att, x, accumulate=True, then=then)
             return
         att = ctx.scratch("att", (T, H * hd), self.dtype)
-        self._attend(ctx, q, k_cache, v_cache, att, tables, sink=self.sink, gate=proj if self.head_gate else None,
-                     gate_offset=gate_off, out_scale=self.out_scale)
+        self._attend(ctx, q, k_cache, v_cache, att, tables, sink=self.sink, out_scale=self.out_scale, gate_dims=gate_dims, **gate)
         self.w_o.forward(att, x, accumulate=True, then=then)
 
     def _attend_maps(self, ctx, q, k_cache, v_cache, tables, x, then) -> None:

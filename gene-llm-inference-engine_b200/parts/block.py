@@ -5,7 +5,7 @@ import torch
 
 from .norm import LayerNorm
 from .registry import FEED_FORWARDS, MIXERS, NORMS, build_part, register_block, sub_weights
-from .stream import EmbeddingMix
+from .stream import EmbeddingAdd, EmbeddingMix
 
 
 @register_block("pre_norm")
@@ -207,7 +207,8 @@ class ParallelBlock:
         self.dtype = build.compute_dtype
         self._next = {}             # run (by the layer whose cache it uses) -> what runs after it, when this kernel can prepare that
 
-    def followed_in_run(self, run, after) -> None:
+    def followed_in_run(self, run, block, stream_input) -> None:
+        after = block if stream_input is None else stream_input
         ok = isinstance(after, EmbeddingMix) or (isinstance(after, ParallelBlock) and
                                                  (hasattr(after.mixer_norm, "scalar") or isinstance(after.mixer_norm, LayerNorm)))
         self._next[run.cache_layer] = after if ok and self._next.get(run.cache_layer, after) is after else None
@@ -297,8 +298,8 @@ class HyperConnectionBlock:
         self.dtype = build.compute_dtype
         self._next = {}             # run (by the layer whose cache it uses) -> the block that runs after it, when of this kind
 
-    def followed_in_run(self, run, block) -> None:
-        ok = isinstance(block, HyperConnectionBlock) and block.streams == self.streams
+    def followed_in_run(self, run, block, stream_input) -> None:
+        ok = stream_input is None and isinstance(block, HyperConnectionBlock) and block.streams == self.streams
         self._next[run.cache_layer] = block if ok else None
 
     def forward(self, ctx, run, x: torch.Tensor) -> None:
@@ -358,6 +359,88 @@ class HyperConnectionBlock:
                 carry["stream_copies"] = (x.data_ptr(), id(nxt))
             else:
                 carry.pop("stream_copies", None)
+
+
+@register_block("sandwich")
+class SandwichBlock:
+    """A norm before and after each sublayer: x <- x + N1'(mixer(N1(x))) and, when the layer has a feed-forward,
+    x <- x + N2'(ff(N2(x))). N1 and N2 are the layer's usual two norms, N1' and N2' its extra parts ``mixer_out_norm`` and
+    ``feed_forward_out_norm`` (a norm that has ``join_stream``).
+
+    The stream x stays 32-bit. A sublayer reads the normed stream in the compute dtype and adds its output to ``y``, which is zero
+    when it starts. What ends a sublayer (``join_stream``, one kernel for norms without a row sum) adds the normed y to x, clears
+    y and writes the normed input of the sublayer that runs next: the feed-forward's, or the next block's mixer's when that block
+    is of this kind; where the embedding's output is added to the stream ahead of it (``EmbeddingAdd``), that is done in the same
+    pass. ``ctx.carry`` tells the next block what it finds."""
+
+    def __init__(self, layer_spec, weights, build):
+        self.mixer_norm = build_part(NORMS, "norm", layer_spec.mixer_norm, sub_weights(weights, "mixer_norm."), build)
+        self.mixer = build_part(MIXERS, "mixer", layer_spec.mixer, sub_weights(weights, "mixer."), build)
+        self.mixer_out_norm = build_extra(layer_spec, "mixer_out_norm", NORMS, "norm", weights, build)
+        self.feed_forward = self.feed_forward_norm = self.feed_forward_out_norm = None
+        if layer_spec.feed_forward is not None:
+            self.feed_forward_norm = build_part(NORMS, "norm", layer_spec.feed_forward_norm,
+                                                sub_weights(weights, "feed_forward_norm."), build)
+            self.feed_forward = build_part(FEED_FORWARDS, "feed-forward", layer_spec.feed_forward,
+                                           sub_weights(weights, "feed_forward."), build)
+            self.feed_forward_out_norm = build_extra(layer_spec, "feed_forward_out_norm", NORMS, "norm", weights, build)
+        self.dtype = build.compute_dtype
+        self._next = {}             # run (by the layer whose cache it uses) -> (the block that runs after it, the stream input ahead of it)
+
+    def followed_in_run(self, run, block, stream_input) -> None:
+        ok = isinstance(block, SandwichBlock) and (stream_input is None or isinstance(stream_input, EmbeddingAdd))
+        self._next[run.cache_layer] = (block, stream_input) if ok else (None, None)
+
+    def forward(self, ctx, run, x: torch.Tensor) -> None:
+        from ..ops import kernels
+        T, D = x.shape
+        y = ctx.scratch("sandwich_y", (T, D), torch.float32)
+        xn = ctx.scratch("normed", (T, D), self.dtype)
+        carry = getattr(ctx, "carry", None)
+        state = carry.get("sandwich") if carry is not None else None
+        # what the block before left: y = 0, and xn = this block's normed input if it is the one it prepared
+        clear = state is not None and state[0] == x.data_ptr()
+        ready = clear and state[1] == id(self)
+        block, stream_input = self._next.get(run.cache_layer, (None, None)) if carry is not None else (None, None)
+        if stream_input is not None and getattr(ctx, "tapping", False):
+            block = stream_input = None         # someone listens to the stream as the layer leaves it
+        second = self.feed_forward is not None
+
+        def after_layer(out_norm):
+            out_norm.join_stream(y, x, None if stream_input is None else stream_input.kept(ctx),
+                                 None if block is None else block.mixer_norm, None if block is None else xn)
+
+        def mixer_half():
+            if not clear:
+                kernels.scale_cast(x, y, None, 0.0)                                   # y = 0
+            if not ready:
+                self.mixer_norm.forward(x, xn)
+            self.mixer.forward(ctx, run, xn, y)
+            if second:
+                self.mixer_out_norm.join_stream(y, x, None, self.feed_forward_norm, xn)
+            else:
+                after_layer(self.mixer_out_norm)
+
+        key = _launch_key(ctx, (self.mixer_norm, None), (self.mixer, run))
+        if key is not None:
+            ctx.recorded(self, ("mixer", run, T, clear, ready) + key, mixer_half)
+        else:
+            mixer_half()
+        ctx.tap("attn_out", run.layer, x)
+        if second:
+            def feed_forward_half():
+                self.feed_forward.forward(ctx, xn, y)
+                after_layer(self.feed_forward_out_norm)
+            key = _launch_key(ctx, (self.feed_forward_norm, None), (self.feed_forward, None))
+            if key is not None:
+                ctx.recorded(self, ("feed_forward", run, T) + key, feed_forward_half)
+            else:
+                feed_forward_half()
+        ctx.tap("ffn_out", run.layer, x)
+        if carry is not None:
+            carry["sandwich"] = (x.data_ptr(), None if block is None else id(block))
+            if stream_input is not None:
+                carry["stream_handed"] = (x.data_ptr(), id(stream_input))
 
 
 def build_extra(layer_spec, key: str, table, what: str, weights, build):

@@ -62,7 +62,8 @@ class SwiGLUFeedForward:
         """Its launches depend on the token count only (which the caller's key holds)."""
         return ()
 
-    def forward(self, ctx, xn: torch.Tensor, x: torch.Tensor) -> None:
+    def forward(self, ctx, xn: torch.Tensor, x: torch.Tensor, accumulate: bool = True) -> None:
+        """``accumulate`` False: x is set to the output instead of being added to."""
         T = xn.shape[0]
         h = ctx.scratch("ffn_hidden", (T, self.intermediate_size), self.dtype)
         if self.dtype is torch.bfloat16 and kernels.gemm_swiglu_supported(T, self.intermediate_size, self.hidden_size):
@@ -75,7 +76,7 @@ class SwiGLUFeedForward:
                 kernels.swiglu(gu, h)
             else:
                 kernels.gated_act(gu, h, self.activation, self.limit, self.b_gate_up)
-        self.w_down.forward(h, x, accumulate=True)
+        self.w_down.forward(h, x, accumulate=accumulate)
         if self.b_down is not None and not self.output_bias_left:
             kernels.add_bias(x, self.b_down)
 
@@ -109,7 +110,7 @@ class UngatedFeedForward:
     def launch_key(self, ctx):
         return ()
 
-    def forward(self, ctx, xn: torch.Tensor, x: torch.Tensor) -> None:
+    def forward(self, ctx, xn: torch.Tensor, x: torch.Tensor, accumulate: bool = True) -> None:
         h = ctx.scratch("ffn_hidden", (xn.shape[0], self.intermediate_size), self.dtype)
         if self.dtype is torch.bfloat16 and self.hidden_size % 8 == 0:
             kernels.gemm_tc(xn, self.w_up.weight, h, w_tiles=self.w_up.weight_tiles, act=self.activation)
@@ -117,7 +118,7 @@ class UngatedFeedForward:
             z = ctx.scratch("ffn_up", (xn.shape[0], self.intermediate_size), torch.float32)
             self.w_up.forward(xn, z)
             kernels.plain_act(z, h, self.activation)
-        self.w_down.forward(h, x, accumulate=True)
+        self.w_down.forward(h, x, accumulate=accumulate)
 
 
 @register_feed_forward("routed_experts")
@@ -131,10 +132,14 @@ class RoutedExpertsFeedForward:
 
     ``scores`` = "softmax": s = softmax(z) over all experts; ``renormalise``: the chosen s_e are divided by their sum
     (+ 1e-20); ``router_scale``: a constant on the weights. ``gated`` False: an expert is W_down,e act(W_up,e u) with
-    ``activation`` one of ``kernels.PLAIN_ACTIVATIONS`` (and so is the shared one).
+    ``activation`` one of ``kernels.PLAIN_ACTIVATIONS`` (and so is the shared one). ``weigh_input``: the weight scales what the
+    expert reads, not what it returns: x += sum over the chosen e of expert_e(s_e u). ``shared_gate``: the shared expert's output
+    is multiplied by sigmoid(w_g u), one number per token (``shared_gate`` [1, hidden], in 32-bit like the router); it is then
+    stored by itself and joins the sum where the experts' outputs do.
 
     Params: ``hidden_size``, ``intermediate_size`` (of one expert), ``experts``, ``top`` and optionally ``activation``
-    ("silu") with ``activation_limit``, ``router`` ("scored", the default, or "table", then with ``vocab_size``), ``shared``.
+    ("silu") with ``activation_limit``, ``router`` ("scored", the default, or "table", then with ``vocab_size``), ``shared`` and
+    the options above.
     Weights: ``router`` [E, hidden] and ``correction`` [E] (scored) or ``table`` [vocab, top] integers, ``w_gate_up``
     [E, 2I, hidden] (an expert's gate rows, then its up rows; not gated: ``w_up`` [E, I, hidden]), ``w_down`` [E, hidden, I],
     the shared expert's under ``shared.``. The ``correction`` may be absent (no correction).
@@ -169,6 +174,7 @@ class RoutedExpertsFeedForward:
         if self.scores not in ("sigmoid", "softmax"):
             raise ValueError(f"routed experts: unknown scores '{self.scores}' (known: sigmoid, softmax)")
         self.renormalise, self.router_scale = bool(params.get("renormalise", False)), float(params.get("router_scale", 1.0))
+        self.weigh_input = bool(params.get("weigh_input", False))
         E, I, D = self.experts, self.intermediate_size, self.hidden_size
         chooser = (("router", (E, D)),) if self.routing == "scored" else (("table", (int(params["vocab_size"]), self.top)),)
         if self.routing == "scored" and "correction" in weights:
@@ -198,6 +204,11 @@ class RoutedExpertsFeedForward:
         if params.get("shared"):
             kind = SwiGLUFeedForward if self.gated else UngatedFeedForward
             self.shared = kind(params["shared"], sub_weights(weights, "shared."), build)
+        self.shared_gate = None
+        if params.get("shared_gate"):
+            if self.shared is None or self.routing != "scored" or weights["shared_gate"].numel() != D:
+                raise ValueError("routed experts: a shared expert's gate needs the shared expert, scored routing and a weight per input")
+            self.shared_gate = weights["shared_gate"].reshape(-1).to(device=dev, dtype=torch.float32).contiguous()
         self.w_first = weights[first[0]].to(device=dev, dtype=dt).contiguous()
         self.w_down = weights["w_down"].to(device=dev, dtype=dt).contiguous()
         self.dtype = dt
@@ -222,12 +233,11 @@ class RoutedExpertsFeedForward:
         n_tiles = ctx.scratch("route_n_tiles", (1,), torch.int32, capacity=1)
         self._route(ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles)
         hidden = ctx.scratch("expert_hidden", (T * top, I), torch.float32, capacity=max(most, T) * top)
-        kernels.expert_product(xn, top, self.w_first, hidden, sorted_rows, tile_group, n_tiles, **self._first_form())
+        kernels.expert_product(xn, top, self.w_first, hidden, sorted_rows, tile_group, n_tiles,
+                               scales=weights if self.weigh_input else None, **self._first_form())
         part = ctx.scratch("expert_out", (T * top, D), torch.float32, capacity=max(most, T) * top)
         kernels.expert_product(hidden, 1, self.w_down, part, sorted_rows, tile_group, n_tiles)
-        kernels.route_combine(part, weights, x)
-        if self.shared is not None:
-            self.shared.forward(ctx, xn, x)
+        self._combine(ctx, xn, part, weights, x)
 
     def _route(self, ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles, **tiles) -> None:
         """The step's (token, choice) pairs and their weights, bucketed by expert."""
@@ -235,8 +245,22 @@ class RoutedExpertsFeedForward:
             kernels.route_table(ctx.tokens, ctx.feedback, self.table, self.experts, ids, weights, sorted_rows, tile_group, n_tiles,
                                 **tiles)
         else:
+            gate = {}
+            if self.shared_gate is not None:
+                gate = {"gate_w": self.shared_gate, "gate_out": ctx.scratch("shared_gate", (xn.shape[0],), torch.float32)}
             kernels.route(xn, self.router, self.correction, self.top, ids, weights, sorted_rows, tile_group, n_tiles,
-                          scores=self.scores, renormalise=self.renormalise, factor=self.router_scale, **tiles)
+                          scores=self.scores, renormalise=self.renormalise, factor=self.router_scale, **gate, **tiles)
+
+    def _combine(self, ctx, xn, part, weights, x, pair_row=None) -> None:
+        """The experts' outputs, and the shared one's, into x."""
+        more = {}
+        if self.shared_gate is not None:
+            out = ctx.scratch("shared_out", tuple(x.shape), torch.float32)
+            self.shared.forward(ctx, xn, out, accumulate=False)
+            more = {"more": out, "more_gate": ctx.scratch("shared_gate", (xn.shape[0],), torch.float32)}
+        kernels.route_combine(part, None if self.weigh_input else weights, x, pair_row=pair_row, top=self.top, **more)
+        if self.shared is not None and self.shared_gate is None:
+            self.shared.forward(ctx, xn, x)
 
     def _first_form(self) -> dict:
         """What the experts' first product does besides multiplying."""
@@ -255,11 +279,9 @@ class RoutedExpertsFeedForward:
         n_tiles = ctx.scratch("route_n_tiles", (1,), torch.int32, capacity=1)
         self._route(ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles, tile_rows=tm, pair_row=pair_row)
         rows = ctx.scratch("expert_rows", (tiles * tm, D), self.dtype, capacity=most_tiles * tm)
-        kernels.gather_rows(xn, top, sorted_rows, n_tiles, tm, rows)
+        kernels.gather_rows(xn, top, sorted_rows, n_tiles, tm, rows, scales=weights if self.weigh_input else None)
         hidden = ctx.scratch("expert_hidden_tc", (tiles * tm, I), self.dtype, capacity=most_tiles * tm)
         kernels.expert_product_tc(rows, self.w_first, hidden, tile_group, n_tiles, **self._first_form())
         part = ctx.scratch("expert_out_tc", (tiles * tm, D), torch.float32, capacity=most_tiles * tm)
         kernels.expert_product_tc(hidden, self.w_down, part, tile_group, n_tiles)
-        kernels.route_combine(part, weights, x, pair_row=pair_row)
-        if self.shared is not None:
-            self.shared.forward(ctx, xn, x)
+        self._combine(ctx, xn, part, weights, x, pair_row)

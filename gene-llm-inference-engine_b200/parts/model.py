@@ -72,12 +72,12 @@ class DecoderModel:
             self.stream_input = build_part(STREAM_INPUTS, "stream input", spec.stream_input,
                                            sub_weights(params, "stream_input."), build)
         self.final_norm = build_part(NORMS, "norm", spec.final_norm, sub_weights(params, "final_norm."), build)
-        # a block may prepare what the block of the next run (or the stream input ahead of it) reads: it is told, run by run,
+        # a block may prepare what the block of the next run (and the stream input ahead of it) reads: it is told, run by run,
         # who follows
         for run, after in zip(self.runs, self.runs[1:]):
             follows = getattr(self.layers[run.layer], "followed_in_run", None)
             if follows is not None:
-                follows(run, self.stream_input if after.stream_input else self.layers[after.layer])
+                follows(run, self.layers[after.layer], self.stream_input if after.stream_input else None)
         if spec.tie_word_embeddings:
             self.head = Linear.over(self.embedding, tiles=weight_tiles)   # the table itself, not a second row-major copy
         else:

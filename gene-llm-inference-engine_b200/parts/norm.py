@@ -36,6 +36,14 @@ class RMSNorm:
         kernels.rmsnorm(x, self.weight, out, self.eps, rows)
         return out
 
+    def join_stream(self, y: torch.Tensor, x: torch.Tensor, more=None, next_norm=None, xn_out=None) -> None:
+        """x += N(y) (+ ``more``), y = 0 and xn_out = next_norm(x): the end of a sublayer whose output is normed."""
+        kernels.add_normed(y, self.weight, x, self.eps, clear_y=True)
+        if more is not None:
+            kernels.add_stream(x, more)
+        if next_norm is not None:
+            next_norm.forward(x, xn_out)
+
 
 @register_norm("rmsnorm_scalar")
 class ScalarRMSNorm(RMSNorm):
@@ -75,3 +83,39 @@ class LayerNorm:
     def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         kernels.layer_norm(x, self.weight, self.bias, out, self.eps, rows)
         return out
+
+
+@register_norm("dynamic_tanh")
+class DynamicTanhNorm:
+    """out = tanh(alpha * x) * weight + bias with one learned number alpha, computed in 32-bit from the 32-bit residual stream; no
+    mean and no variance is taken. Params: ``size``. Weights: ``weight`` and ``bias`` [size], ``alpha`` (one value, any shape)."""
+
+    def __init__(self, params, weights, build):
+        self.size = int(params["size"])
+        for name in ("weight", "bias"):
+            w = weights[name]
+            if tuple(w.shape) != (self.size,):
+                raise ValueError(f"dynamic_tanh: {name} has shape {tuple(w.shape)}, expected ({self.size},)")
+            setattr(self, name, w.to(device=build.device, dtype=torch.float32).contiguous())
+        if weights["alpha"].numel() != 1:
+            raise ValueError(f"dynamic_tanh: alpha has {weights['alpha'].numel()} values, expected one")
+        self.alpha = float(weights["alpha"].float())
+
+    @property
+    def constants(self):
+        return self.alpha, self.weight, self.bias
+
+    def launch_key(self, ctx):
+        """Its one launch depends on the number of rows only (which the caller's key holds)."""
+        return ()
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        kernels.dynamic_tanh(x, self.alpha, self.weight, self.bias, out, rows)
+        return out
+
+    def join_stream(self, y: torch.Tensor, x: torch.Tensor, more=None, next_norm=None, xn_out=None) -> None:
+        """x += N(y) (+ ``more``), y = 0 and xn_out = next_norm(x): one pass where the next norm is of this kind too."""
+        fused = isinstance(next_norm, DynamicTanhNorm)
+        kernels.add_dynamic_tanh(y, self.constants, x, more, next_norm.constants if fused else None, xn_out if fused else None, clear_y=True)
+        if next_norm is not None and not fused:
+            next_norm.forward(x, xn_out)

@@ -87,6 +87,8 @@ class RotaryOnDevice:
     and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), pair i turns at f_i (1 - r_i) + f_i r_i / factor, and
     cos and sin are multiplied by ``amplitude`` = 0.1 ln(factor) + 1 (1 without scaling).
 
+    Optional ``linear_scaling`` {factor}: every pair turns at f / factor.
+
     Optional ``wavelength_scaling`` {factor, low, high, original}: a pair whose wavelength 2 pi / f is shorter than
     original / high keeps f, one whose wavelength is longer than original / low turns at f / factor, and between the two
     f (1 - s) / factor + f s with s = (original / wavelength - low) / (high - low) (the frequencies of ``rope_frequencies``
@@ -123,10 +125,14 @@ class RotaryOnDevice:
             r = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
             freq = freq / factor * r + freq * (1.0 - r)
             self.amplitude = 0.1 * math.log(factor) + 1.0
-        wave = params.get("wavelength_scaling")
+        linear, wave = params.get("linear_scaling"), params.get("wavelength_scaling")
+        if sum(map(bool, (ramp, linear, wave))) > 1:
+            raise ValueError("rope: ramp_scaling, linear_scaling and wavelength_scaling exclude one another")
+        if linear:
+            if not float(linear["factor"]) > 0:
+                raise ValueError("rope: the factor of linear_scaling must be positive")
+            freq = freq / float(linear["factor"])
         if wave:
-            if ramp:
-                raise ValueError("rope: ramp_scaling and wavelength_scaling exclude one another")
             freq = rope_frequencies(self.head_dim, float(params["theta"]), {
                 "factor": wave["factor"], "low_freq_factor": wave["low"], "high_freq_factor": wave["high"],
                 "original_max_position": wave["original"]}, self.rotary_dim, round_theta=False)

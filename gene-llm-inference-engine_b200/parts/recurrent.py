@@ -44,11 +44,13 @@ class LinearAttentionMixer:
     lambda_h the head's factor:  q = phi(Wq u), k = phi(Wk u) (H heads of dk), v = phi(Wv u) (H heads of dv);
     M_t = lambda_h M_(t-1) + k_t (x) v_t  (a dk x dv matrix per head, (x) the outer product);  y_t = M_t^T q_t, unscaled.
     All heads' y side by side are brought to unit RMS as one vector, weighted by ``norm`` [H dv], gated elementwise
-    by sigmoid(Wg u) and sent through ``w_o``.
+    by sigmoid(Wg u) and sent through ``w_o``. Options: ``query_scale``, a constant on the queries (what a constant on the
+    keys comes to); ``norm_per_head``: each head's y is brought to unit RMS on its own; ``norm_weights`` False: the norm has
+    no weights; ``gate`` "silu": the gate is SiLU(Wg u).
 
     Params: ``hidden_size``, ``num_heads``, ``key_dim``, ``value_dim``, ``decay`` (lambda, one per head), ``norm_eps``,
-    ``activation`` ("silu" or "none") and optionally ``out_scale``. Weights: ``w_in`` [(2 H dk + 2 H dv), hidden]
-    (rows of Wq, Wk, Wv, Wg in this order), ``w_o`` [hidden, H dv], ``norm`` [H dv]."""
+    ``activation`` ("silu" or "none") and optionally ``out_scale`` and the options above. Weights: ``w_in``
+    [(2 H dk + 2 H dv), hidden] (rows of Wq, Wk, Wv, Wg in this order), ``w_o`` [hidden, H dv], ``norm`` [H dv]."""
 
     graph_safe = True
 
@@ -60,6 +62,11 @@ class LinearAttentionMixer:
         if params.get("activation", "silu") not in ("silu", "none"):
             raise ValueError(f"linear attention: unknown activation '{params.get('activation')}'")
         self.out_scale = float(params.get("out_scale", 1.0))
+        self.q_scale = float(params.get("query_scale", 1.0))
+        self.norm_groups = self.num_heads if params.get("norm_per_head") else 1
+        self.gate_act = params.get("gate", "sigmoid")
+        if self.gate_act not in ("sigmoid", "silu"):
+            raise ValueError(f"linear attention: unknown gate '{self.gate_act}'")
         decay = [float(d) for d in params["decay"]]
         if len(decay) != self.num_heads:
             raise ValueError("linear attention: one decay per head is needed")
@@ -74,7 +81,10 @@ class LinearAttentionMixer:
             raise ValueError(f"linear attention: w_o has shape {tuple(weights['w_o'].shape)}, expected ({D}, {H * dv})")
         self.w_in = Linear(weights["w_in"], build.compute_dtype, build.device, tiles=build.weight_tiles)
         self.w_o = Linear(weights["w_o"], build.compute_dtype, build.device, tiles=build.weight_tiles)
-        self.norm = _vector(weights, "norm", H * dv, build, "linear attention")
+        if params.get("norm_weights", True):
+            self.norm = _vector(weights, "norm", H * dv, build, "linear attention")
+        else:
+            self.norm = torch.ones(H * dv, dtype=torch.float32, device=build.device)
         self.dtype = build.compute_dtype
         self.state_offset = 0
 
@@ -97,10 +107,10 @@ class LinearAttentionMixer:
         o = ctx.scratch("lin_att_out", (T, H * dv), torch.float32)
         kernels.linear_scan(proj, 0, proj, H * dk, proj, 2 * H * dk, H, 1, dk, dv, self.activate,
                             ctx.state(run.cache_layer), self.state_offset, ctx.seg_start, ctx.seg_len, ctx.state_slots, o, decay=self.decay,
-                            **_scan_workspaces(ctx, T, H, dk, dv))
+                            q_scale=self.q_scale, **_scan_workspaces(ctx, T, H, dk, dv))
         y = ctx.scratch("lin_att_normed", (T, H * dv), self.dtype)
-        kernels.gated_group_norm(o, proj, 2 * H * dk + H * dv, self.norm, y, 1, self.eps, gate_first=False,
-                                 out_scale=self.out_scale)
+        kernels.gated_group_norm(o, proj, 2 * H * dk + H * dv, self.norm, y, self.norm_groups, self.eps, gate_first=False,
+                                 out_scale=self.out_scale, gate_act=self.gate_act)
         self.w_o.forward(y, x, accumulate=True, then=then)
 
 

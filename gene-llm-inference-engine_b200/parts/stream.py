@@ -57,3 +57,28 @@ class EmbeddingMix:
                 kernels.take_stream(x, start, taken)
             self.w_x.forward(taken, x, accumulate=True)
         ctx.recorded(self, ("pass", ctx.n_tokens, handed), launch)
+
+
+@register_stream_input("embedding_add")
+class EmbeddingAdd:
+    """x <- x + x0 with x0 the embedding's output, which is kept when a step begins. The kernel that ends the layer before may
+    add it in its own pass (``kept``, ``ctx.carry``). Params: ``hidden_size``."""
+
+    graph_safe = True
+
+    def __init__(self, params, weights, build):
+        self.hidden_size = int(params["hidden_size"])
+
+    def kept(self, ctx) -> torch.Tensor:
+        """x0 [T, hidden] 32-bit."""
+        return ctx.scratch("stream_start", (ctx.n_tokens, self.hidden_size), torch.float32)
+
+    def begin(self, ctx, x: torch.Tensor) -> None:
+        x0 = self.kept(ctx)
+        ctx.recorded(self, ("begin", ctx.n_tokens), lambda: kernels.scale_cast(x, x0, None, 1.0))
+
+    def forward(self, ctx, x: torch.Tensor) -> None:
+        if ctx.carry.pop("stream_handed", None) == (x.data_ptr(), id(self)):
+            return                      # added by the kernel that ended the layer before
+        x0 = self.kept(ctx)
+        ctx.recorded(self, ("pass", ctx.n_tokens), lambda: kernels.add_stream(x, x0))

@@ -437,6 +437,93 @@ def mimolix_weight_plan(cfg) -> WeightPlan:
     return WeightPlan(rules, [], assemble)
 
 
+def kidarax_weight_plan(cfg) -> WeightPlan:
+    """Tensor names and shapes of a Kidarax checkpoint: ``embed`` (also the head), ``final.norm`` and, for layer i, the norms
+    ``l<i>.norm1`` and ``l<i>.norm1b`` (with a feed-forward also ``norm2``, ``norm2b``), the mixer's tensors under ``l<i>.mix.`` and
+    the feed-forward's under ``l<i>.mlp.`` (dense: ``up``, ``down``; a mixture: ``e<k>.gate`` / ``.up`` / ``.down`` per expert,
+    ``router``, ``shared.gate`` / ``.up`` / ``.down`` and ``shared.sg``). A norm is three tensors: the weight, ``.b`` and the number
+    ``.alpha``. Projections that read the same input become one product: [q; k; v; g] of a retention mixer or an attention,
+    [q; dkv; g] of the latent attention, [gate; up] of an expert; the experts' matrices are stacked."""
+    D, V = cfg.width, cfg.vocab
+    rules = [TensorRule("embed", (V, D))]
+
+    def norm(name: str) -> List[TensorRule]:
+        return [TensorRule(name, (D,), "vector"), TensorRule(name + ".b", (D,), "vector", (0.0, 0.05)),
+                TensorRule(name + ".alpha", (), "vector", ("uniform", 0.4, 1.2))]
+
+    for i, layer in enumerate(cfg.layers):
+        p, m = f"l{i}.", layer.mixer
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if layer.mlp is not None else ()):
+            rules += norm(p + n)
+        q = p + "mix."
+        if layer.type == "retention":
+            rules += [TensorRule(q + "q", (m.heads * m.dim, D)), TensorRule(q + "k", (m.heads * m.dim, D)),
+                      TensorRule(q + "v", (m.heads * m.vdim, D)), TensorRule(q + "g", (m.heads * m.vdim, D))]
+        elif layer.type == "attention":
+            for n, rows in (("q", m.heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
+                rules += [TensorRule(q + n, (rows, D)), TensorRule(q + n + ".b", (rows,), "vector", (0.0, 0.1))]
+            rules.append(TensorRule(q + "g", (m.heads * m.vdim, D)))
+        else:
+            rules += [TensorRule(q + "q", (m.heads * (m.dim + m.rot_dim), D)), TensorRule(q + "dkv", (m.kv_rank + m.rot_dim, D)),
+                      TensorRule(q + "dkv.norm", (m.kv_rank,), "vector"), TensorRule(q + "uk", (m.heads * m.dim, m.kv_rank)),
+                      TensorRule(q + "uv", (m.heads * m.vdim, m.kv_rank)), TensorRule(q + "sink", (m.heads,), "vector", (0.0, 1.0)),
+                      TensorRule(q + "g", (m.heads, D))]
+        rules.append(TensorRule(q + "o", (D, m.heads * m.vdim)))
+        f, q = layer.mlp, p + "mlp."
+        if f is None:
+            continue
+        if not hasattr(f, "experts"):
+            rules += [TensorRule(q + "up", (f.ff, D)), TensorRule(q + "down", (D, f.ff))]
+            continue
+        for part, ff in [(f"e{e}", f.ff) for e in range(f.experts)] + ([("shared", f.shared_ff)] if f.shared_ff is not None else []):
+            rules += [TensorRule(f"{q}{part}.gate", (ff, D)), TensorRule(f"{q}{part}.up", (ff, D)), TensorRule(f"{q}{part}.down", (D, ff))]
+        rules.append(TensorRule(q + "router", (f.experts, D)))
+        if f.shared_ff is not None:
+            rules.append(TensorRule(q + "shared.sg", (1, D)))
+    rules += norm("final.norm")
+
+    def assemble(t: Dict[str, torch.Tensor]) -> Dict[str, torch.Tensor]:
+        out: Dict[str, torch.Tensor] = {"embedding.weight": t["embed"], "head.weight": t["embed"]}
+
+        def take_norm(part: str, name: str) -> None:
+            out[part + ".weight"], out[part + ".bias"], out[part + ".alpha"] = t[name], t[name + ".b"], t[name + ".alpha"]
+
+        take_norm("final_norm", "final.norm")
+        for i, layer in enumerate(cfg.layers):
+            p, q = f"l{i}.", f"layers.{i}."
+            take_norm(q + "mixer_norm", p + "norm1")
+            take_norm(q + "mixer_out_norm", p + "norm1b")
+            a, b = p + "mix.", q + "mixer."
+            if layer.type == "retention":
+                out[b + "w_in"] = _cat([t[a + n] for n in ("q", "k", "v", "g")])
+            elif layer.type == "attention":
+                out[b + "w_qkv"] = _cat([t[a + n] for n in ("q", "k", "v", "g")])
+                out[b + "b_qkv"] = _cat([t[a + n + ".b"] for n in ("q", "k", "v")])
+            else:
+                out[b + "w_down"] = _cat([t[a + n] for n in ("q", "dkv", "g")])
+                out[b + "kv_latent_norm"], out[b + "sink"] = t[a + "dkv.norm"], t[a + "sink"]
+                out[b + "w_uk"], out[b + "w_uv"] = t[a + "uk"], t[a + "uv"]
+            out[b + "w_o"] = t[a + "o"]
+            f = layer.mlp
+            if f is None:
+                continue
+            take_norm(q + "feed_forward_norm", p + "norm2")
+            take_norm(q + "feed_forward_out_norm", p + "norm2b")
+            a, b = p + "mlp.", q + "feed_forward."
+            if not hasattr(f, "experts"):
+                out[b + "w_up"], out[b + "w_down"] = t[a + "up"], t[a + "down"]
+                continue
+            out[b + "w_gate_up"] = torch.stack([_cat([t[f"{a}e{e}.gate"], t[f"{a}e{e}.up"]]) for e in range(f.experts)])
+            out[b + "w_down"] = torch.stack([t[f"{a}e{e}.down"] for e in range(f.experts)])
+            out[b + "router"] = t[a + "router"]
+            if f.shared_ff is not None:
+                out[b + "shared.w_gate_up"] = _cat([t[a + "shared.gate"], t[a + "shared.up"]])
+                out[b + "shared.w_down"], out[b + "shared_gate"] = t[a + "shared.down"], t[a + "shared.sg"]
+        return out
+
+    return WeightPlan(rules, [], assemble)
+
+
 def _cat(parts: List[torch.Tensor]) -> torch.Tensor:
     """Concatenates rows; parts of different stored dtypes are widened to 32-bit first."""
     if len({p.dtype for p in parts}) > 1:
