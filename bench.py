@@ -8,6 +8,7 @@
     python bench.py --scenario nipadra               (the Nipadra design beside Llama at equal layer sizes, see run_nipadra)
     python bench.py --scenario gekupel               (the Gekupel design beside Llama at equal layer sizes, see run_gekupel)
     python bench.py --scenario pinorax               (the Pinorax design beside Gekupel and Llama at equal layer sizes, see run_pinorax)
+    python bench.py --scenario kidarax               (the Kidarax design beside Nipadra, Pinorax and Llama at equal layer sizes, see run_kidarax)
     python bench.py --scenario mimolix               (the Mimolix design beside Pinorax, Fovezen and Llama at equal layer sizes, see run_mimolix)
     python bench.py --scenario fovezen               (the Fovezen design beside Nipadra and Llama at equal layer sizes, see run_fovezen)
 
@@ -1457,6 +1458,250 @@ def run_mimolix(args):
     return 0
 
 
+# ---------------------------------------------------------------------------------------------- Kidarax beside Nipadra and Pinorax
+def kidarax_config(width, ff, layers, vocab, heads, head_dim, kv_heads):
+    """A Kidarax model with the layer sizes of a Llama shape. Layers in turn: retention (width / 128 heads of 128 x 128) with a
+    dense squared-ReLU feed-forward of 3/2 of the gated width (as many multiply-adds), attention (Llama's heads), latent
+    attention (the heads and the latent of ``pinorax_config``, half a head more of rotated keys), retention; all but the first
+    with the mixture of ``pinorax_config``. One pass."""
+    lh = width // 128
+    decay = [1.0 - 2.0 ** (-5 - 3 * i / max(1, lh - 1)) for i in range(lh)]
+    ret = {"heads": lh, "dim": 128, "vdim": 128, "decay": decay}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+           "rot": {"base": 500000.0, "dims": head_dim, "scaling": {"factor": 4.0}}}
+    rot = head_dim // 2
+    lat = {"heads": max(heads // 2, 1), "dim": head_dim, "rot_dim": rot, "vdim": head_dim, "kv_rank": min(512, width // 4),
+           "scale": (head_dim + rot) ** -0.5,
+           "rot": {"base": 500000.0, "dims": rot, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    moe = {"expert": {"ff": 3 * ff // 8}, "kind": "moe", "router": {"experts": 8, "top": 2}, "shared": {"ff": ff // 4}}
+    kinds = [("retention", ret, {"ff": 3 * ff // 2, "kind": "dense"}), ("attention", att, moe), ("latent_attention", lat, moe), ("retention", ret, moe)]
+    return {"architecture": "Kidarax", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": kinds[i % 4][2]} for i in range(layers)]}
+
+
+def kidarax_kernel_table(width, ff, heads, head_dim, kv_heads, T, pk):
+    """Each kernel that the Kidarax design added or changed, alone, beside the like kernel of another design's path, at the sizes of
+    one layer: a prompt portion of ``T`` tokens of one request and a decode step of 8 requests at a context of ``T``. ``frac``
+    is the time the kernel's algorithmic bytes (or, where larger, its multiply-adds on the tensor cores) need at the measured
+    peaks, divided by the time it took; ``frac_of_32bit_issue`` the same against the CUDA cores' 32-bit rate, for kernels whose
+    arithmetic has to stay 32-bit."""
+    import torch
+    from geneinfer_b200.ops import kernels as K
+    from geneinfer_b200.ops.linear import Linear
+    dev = torch.device("cuda:0")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    rows = []
+    props = torch.cuda.get_device_properties(dev)
+    simt_ops = props.multi_processor_count * 128 * 1.965e9
+    bf = torch.bfloat16
+
+    def add(name, like, fn, nbytes, flops=0.0, simt=0.0):
+        ms = time_calls(fn, flush=flush)
+        ideal = max(nbytes / (pk["hbm_gbs"] * 1e9), flops / (pk["bf16_tflops"] * 1e12)) * 1e3
+        row = {"kernel": name, "like": like, "us": round(ms * 1e3, 1), "frac": round(ideal / ms, 3)}
+        if simt:
+            row["frac_of_32bit_issue"] = round(simt / simt_ops * 1e3 / ms, 3)
+        rows.append(row)
+
+    D, page = width, 16
+    for what, R, n in (("prefill", 1, T), ("decode", 8, 1)):
+        N = R * n
+        i32 = dict(dtype=torch.int32, device=dev)
+        s0, sl, slots = torch.arange(R, **i32) * n, torch.full((R,), n, **i32), torch.arange(R, **i32)
+        rr = torch.arange(R, **i32).repeat_interleave(n)
+        # norms before and after a sublayer
+        x, y, more = (torch.randn(N, D, device=dev) for _ in range(3))
+        xn = torch.empty(N, D, dtype=bf, device=dev)
+        w, b = torch.ones(D, device=dev), torch.zeros(D, device=dev)
+        tn = (0.7, w, b)
+        add(f"add_dynamic_tanh with the next norm ({what})", "depth_mix", lambda: K.add_dynamic_tanh(y, tn, x, None, tn, xn, clear_y=True), N * D * 18)
+        add(f"add_dynamic_tanh with the embedding's output and the next norm ({what})", "depth_mix",
+            lambda: K.add_dynamic_tanh(y, tn, x, more, tn, xn, clear_y=True), N * D * 22)
+        add(f"depth_mix with the next layer norm, Mimolix ({what})", "", lambda: K.depth_mix(x, y, 0.5, next_weight=w, next_bias=b, eps=1e-6, xn_out=xn), N * D * 18)
+        add(f"add_normed, Gekupel ({what})", "", lambda: K.add_normed(y, w, x, 1e-6, xn_out=xn, clear_y=True), N * D * 18)
+        add(f"dynamic_tanh ({what})", "layer_norm", lambda: K.dynamic_tanh(x, *tn, xn), N * D * 6)
+        add(f"layer_norm, Mimolix ({what})", "", lambda: K.layer_norm(x, w, b, xn, 1e-6), N * D * 6)
+        add(f"add_stream ({what})", "take_stream", lambda: K.add_stream(x, more), N * D * 12)
+        add(f"take_stream, Mimolix ({what})", "", lambda: K.take_stream(x, more, xn), N * D * 14)
+        # retention: the recurrence of linear attention, the norm per head and its gate
+        H, dk, dv = D // 128, 128, 128
+        proj = torch.randn(N, 2 * H * dk + 2 * H * dv, device=dev) * 0.5
+        state, out = torch.zeros(R, H * dk * dv, device=dev), torch.empty(N, H * dv, device=dev)
+        decay = torch.full((H,), 0.99, device=dev)
+        parts = {}
+        if N > K.SCAN_PART:
+            parts = {"part_len": K.SCAN_PART, "ws_state": torch.empty(K.scan_parts(N, R), H * dk * dv, device=dev), "ws_decay": torch.empty(N, H, device=dev)}
+        for name, like, act in ((f"linear_scan, no activation, scaled queries ({what})", "linear_scan", False), (f"linear_scan, SiLU, Nipadra ({what})", "", True)):
+            add(name, like, lambda: K.linear_scan(proj, 0, proj, H * dk, proj, 2 * H * dk, H, 1, dk, dv, act, state, 0, s0, sl, slots, out, decay=decay,
+                                                  q_scale=1.0 if act else 0.09, **parts),
+                N * (2 * H * dk + 2 * H * dv) * 4 + 2 * R * H * dk * dv * 4, simt=N * H * dk * dv * (4.0 if parts else 3.0))
+        yb, nw = torch.empty(N, H * dv, dtype=bf, device=dev), torch.ones(H * dv, device=dev)
+        add(f"gated_group_norm per head, SiLU gate after ({what})", "gated_group_norm",
+            lambda: K.gated_group_norm(out, proj, 2 * H * dk + H * dv, nw, yb, H, 1e-6, False, gate_act="silu"), N * H * dv * 10)
+        add(f"gated_group_norm, Nipadra ({what})", "", lambda: K.gated_group_norm(out, proj, 2 * H * dk + H * dv, nw, yb, 1, 1e-6, False), N * H * dv * 10)
+        # attention: biases before the rotation, a gate per value in the last step
+        A, C = heads * head_dim, (heads + 2 * kv_heads) * head_dim
+        ap = torch.randn(N, C + A, device=dev)
+        bias = torch.randn(C + A, device=dev)
+        n_pages = R * ((T + page - 1) // page)
+        kc, vc = (torch.randn(n_pages, kv_heads, page, head_dim, device=dev).to(bf) for _ in range(2))
+        tables = torch.arange(n_pages, **i32).view(R, -1)
+        pos = (torch.arange(n, **i32) + (T - n)).repeat(R)
+        q, att = torch.empty(N, A, dtype=bf, device=dev), torch.empty(N, A, dtype=bf, device=dev)
+        freq, hw = torch.rand(head_dim // 2, device=dev), torch.ones(head_dim, device=dev)
+        add(f"norm_rope_store with biases ({what})", "norm_rope_store", lambda: K.norm_rope_store(
+            ap, 0, A, A + kv_heads * head_dim, None, None, 0.0, freq, False, pos, rr, tables, q, kc, vc, heads, kv_heads, head_dim, page, bias=bias), N * C * 6)
+        add(f"norm_rope_store, norm per head, Nipadra ({what})", "", lambda: K.norm_rope_store(
+            ap, 0, A, A, hw, hw, 1e-6, freq, True, pos, rr, tables, q, kc, vc, heads, kv_heads, head_dim, page), N * C * 6)
+        seen = sum(p + 1 for p in range(T - n, T))
+        cache_bytes = R * T * kv_heads * head_dim * 4
+        rows_dec = torch.arange(R, **i32)
+        per_tile = 128 // (heads // kv_heads)
+        work = torch.tensor([(t, min(per_tile, n - t), 0) for t in range(0, n, per_tile)][::-1], **i32)
+        chunk = K.attention_chunk_keys()
+        n_chunks = (T + chunk - 1) // chunk
+        part_o, part_ml = torch.empty(R, heads * n_chunks * head_dim, device=dev), torch.empty(R, heads * n_chunks * 2, device=dev)
+
+        def attend(**ep):
+            if n == 1:
+                K.attention_decode(q, kc, vc, att, rows_dec, rr, pos, tables, heads, kv_heads, head_dim, page, 0.1, None, part_o, part_ml, n_chunks, n_chunks, **ep)
+            else:
+                K.attention_prefill_tc(q, kc, vc, att, work, pos, tables, heads, kv_heads, head_dim, page, 0.1, None, **ep)
+        add(f"attention, a gate per value ({what})", "attention", lambda: attend(gate=ap, gate_offset=C, gate_dims=head_dim), cache_bytes + N * A * 8,
+            4.0 * R * seen * A)
+        add(f"attention, a gate per head, Nipadra's form ({what})", "", lambda: attend(gate=ap, gate_offset=C), cache_bytes + N * A * 4, 4.0 * R * seen * A)
+
+        class Ctx:                      # what attention_rows_of_step reads of a step
+            row_req, positions, page_size, max_position, kept = rr, pos, page, T, {}
+
+            @staticmethod
+            def scratch(name, shape, dtype, capacity=None):
+                key = (name, tuple(shape), dtype)
+                if key not in Ctx.kept:
+                    Ctx.kept[key] = torch.empty(shape, dtype=dtype, device=dev)
+                return Ctx.kept[key]
+
+            @staticmethod
+            def attention_work(per_tile):
+                if n == 1:
+                    return rows_dec, work[:0], T
+                return rows_dec[:0], torch.tensor([(t, min(per_tile, n - t), 0) for t in range(0, n, per_tile)], **i32), 0
+        for name, like, ep in ((f"attention_rows, a gate per value, where other sizes run ({what})", "attention_rows", {"gate": ap, "gate_offset": C}),
+                               (f"attention_rows without a gate, Gekupel ({what})", "", {})):
+            add(name, like, lambda: K.attention_rows_of_step(Ctx, q, kc, vc, att, tables, heads, kv_heads, head_dim, head_dim, 0.1, None, None, None, None, **ep),
+                cache_bytes + N * A * (8 if ep else 4), 4.0 * R * seen * A)
+        # latent attention
+        lh, kr, rot = heads // 2, min(512, width // 4), head_dim // 2
+        cols = lh * (head_dim + rot) + kr + rot + lh
+        down = torch.randn(N, cols + -cols % 8, device=dev)
+        cache = torch.randn(n_pages, 1, page, kr + rot, device=dev).to(bf)
+        wc, fr = torch.ones(kr, device=dev), torch.rand(rot // 2, device=dev)
+        c0 = lh * (head_dim + rot)
+        for name, like, il in ((f"latent_store, pairs of halves ({what})", "latent_store", False), (f"latent_store, neighbouring pairs, Gekupel ({what})", "", True)):
+            add(name, like, lambda: K.latent_store(down, 0, None, None, c0, wc, c0 + kr, fr, 1.2, 1e-6, pos, rr, tables, cache, page, interleaved=il),
+                N * (kr + rot) * 6)
+        wuk = torch.randn(lh, kr, head_dim, device=dev).to(bf)
+        qa = torch.empty(N, lh * (kr + rot), device=dev)
+        for name, like, il in ((f"head_product, queries with a rotated tail of halves ({what})", "head_product", False),
+                               (f"head_product, queries with a rotated tail of neighbours, Gekupel ({what})", "", True)):
+            add(name, like, lambda: K.head_product(down, 0, head_dim + rot, wuk, qa, 0, kr + rot, tail=rot, freq=fr, amplitude=1.2, positions=pos, interleaved=il),
+                lh * kr * head_dim * 2 + N * lh * (head_dim + kr + 2 * rot) * 4, simt=float(N * lh * kr * head_dim))
+        ol, lsink = torch.empty(N, lh * kr, device=dev), torch.zeros(lh, device=dev)
+        add(f"attention_rows over the latent and the rotated part, sink (unchanged) ({what})", "", lambda: K.attention_rows_of_step(
+            Ctx, qa, cache, None, ol, tables, lh, 1, kr + rot, kr, 0.1, None, None, None, lsink), R * T * (kr + rot) * 2 + N * lh * (2 * kr + rot) * 4,
+            2.0 * R * seen * lh * (2 * kr + rot))
+        wuv = torch.randn(lh, head_dim, kr, device=dev).to(bf)
+        lat = torch.empty(N, lh * head_dim, dtype=bf, device=dev)
+        gz = torch.randn(N, lh * head_dim, device=dev)
+        add(f"head_product, values with a gate per head ({what})", "head_product", lambda: K.head_product(
+            ol, 0, kr, wuv, lat, 0, head_dim, gate=down, gate_offset=c0 + kr + rot, gate_per_head=True), lh * kr * head_dim * 2 + N * lh * (kr * 4 + head_dim * 2),
+            simt=float(N * lh * kr * head_dim))
+        add(f"head_product, values with a gate per value, Pinorax ({what})", "", lambda: K.head_product(ol, 0, kr, wuv, lat, 0, head_dim, gate=gz),
+            lh * kr * head_dim * 2 + N * lh * (kr * 4 + head_dim * 6), simt=float(N * lh * kr * head_dim))
+        # experts whose weights scale what they read, and the gated shared expert
+        E, top, I, Is = 8, 2, 3 * ff // 8, ff // 4
+        xb = torch.randn(N, D, device=dev).to(bf)
+        router, sg, corr = torch.randn(E, D, device=dev) * 0.02, torch.randn(D, device=dev) * 0.02, torch.zeros(E, device=dev)
+        tc_form = N * top >= 256
+        tm = 128 if tc_form else K.grouped_tile_rows()
+        tiles = K.route_tiles(N, top, E, tm)
+        ids, wts, gate = torch.empty(N, top, **i32), torch.empty(N, top, device=dev), torch.empty(N, device=dev)
+        srt, grp, cnt, prow = torch.empty(tiles * tm, **i32), torch.empty(tiles, **i32), torch.empty(1, **i32), torch.empty(N * top, **i32)
+        add(f"route + bucket with the shared expert's gate ({what})", "route", lambda: K.route(
+            xb, router, None, top, ids, wts, srt, grp, cnt, tile_rows=tm, pair_row=prow, gate_w=sg, gate_out=gate), N * D * 2 + (E + 1) * D * 4)
+        add(f"route + bucket, Gekupel ({what})", "", lambda: K.route(xb, router, corr, top, ids, wts, srt, grp, cnt, tile_rows=tm, pair_row=prow),
+            N * D * 2 + E * D * 4)
+        wg = torch.randn(E, 2 * I, D, device=dev).to(bf) * 0.02
+        used = min(E, N * top)
+        if tc_form:
+            ar, h = torch.empty(tiles * tm, D, dtype=bf, device=dev), torch.empty(tiles * tm, I, dtype=bf, device=dev)
+            for name, like, sc in ((f"gather_rows times the pairs' weights ({what})", "gather_rows", wts), (f"gather_rows, Gekupel ({what})", "", None)):
+                add(name, like, lambda: K.gather_rows(xb, top, srt, cnt, tm, ar, scales=sc), N * D * 2 + N * top * D * 2)
+            add(f"experts' first product, gated SiLU, tensor cores (unchanged) ({what})", "", lambda: K.expert_product_tc(ar, wg, h, grp, cnt, gated="silu"),
+                used * 2 * I * D * 2 + N * top * (D + I) * 2, 4.0 * N * top * I * D)
+        else:
+            h = torch.empty(N * top, I, device=dev)
+            for name, like, sc in ((f"experts' first product times the pairs' weights, tiles of 16 rows ({what})", "experts", wts),
+                                   (f"experts' first product, tiles of 16 rows, Pinorax ({what})", "", None)):
+                add(name, like, lambda: K.expert_product(xb, top, wg, h, srt, grp, cnt, gated="silu", scales=sc), used * 2 * I * D * 2,
+                    simt=float(N * top * 2 * I * D))
+        part = torch.randn(tiles * tm if tc_form else N * top, D, device=dev)
+        pr = prow if tc_form else None
+        add(f"route_combine with the gated shared expert ({what})", "route_combine", lambda: K.route_combine(part, None, y, pr, top=top, more=more, more_gate=gate),
+            N * D * (top * 4 + 12))
+        add(f"route_combine, Gekupel ({what})", "", lambda: K.route_combine(part, wts, y, pr), N * D * (top * 4 + 8))
+        ld = Linear(torch.randn(D, Is) * 0.02, bf, dev)
+        hs = torch.randn(N, Is, device=dev).to(bf)
+        add(f"shared expert's last product, stored ({what})", "gemm", lambda: ld.forward(hs, more), D * Is * 2 + N * (Is * 2 + D * 4), 2.0 * N * Is * D)
+        add(f"shared expert's last product, added, Pinorax ({what})", "", lambda: ld.forward(hs, more, accumulate=True), D * Is * 2 + N * (Is * 2 + D * 8), 2.0 * N * Is * D)
+    return rows
+
+
+def run_kidarax(args):
+    """Prefill (one 2,048-token prompt in one step) and decode (batch 8 at context 2,048) throughput of Kidarax models whose
+    layers have the sizes of the Llama-3.2-1B and Llama-3.1-8B shapes (four layers each, random bf16 weights), beside Nipadra
+    (the closest existing design in its linear attention and its gated attention), Pinorax (the closest in its latent attention
+    and its experts) and Llama models of the same sizes; then every kernel that the design added or changed alone beside its
+    like kernel. One JSON line."""
+    import torch
+    from geneinfer_b200 import Engine
+    from geneinfer_b200.weights import write_random_model
+    pk = peaks()
+    layers = args.layers or 4
+    context, batch, T = 2048, 8, PREFILL_TOKENS
+    models = []
+    for name, base in (("1b", LLAMA_1B), ("8b", LLAMA_8B)):
+        llama = dict(base, num_hidden_layers=layers, tie_word_embeddings=True)
+        width, ff, vocab, heads, hd, kv = (base[k] for k in ("hidden_size", "intermediate_size", "vocab_size", "num_attention_heads", "head_dim",
+                                                             "num_key_value_heads"))
+        pin = pinorax_config(width, ff, layers, vocab, heads, hd, context)
+        nip = nipadra_config(width, ff, layers, vocab, heads, hd, kv, context)
+        for arch, cfg in (("Llama", llama), ("Nipadra", nip), ("Pinorax", pin), ("Kidarax", kidarax_config(width, ff, layers, vocab, heads, hd, kv))):
+            if arch == "Llama":
+                folder = model_folder(cfg)
+            else:
+                folder = os.path.join(tempfile.gettempdir(), f"geneinfer_bench_{arch.lower()}_{name}_{layers}_{context}_{os.getuid()}")
+                if not os.path.isfile(os.path.join(folder, "done")):
+                    write_random_model(cfg, 1, folder, "bfloat16", std=0.02)
+                    open(os.path.join(folder, "done"), "w").close()
+            llm = Engine(folder, dtype="bfloat16", max_seq_len=context, page_size=PAGE, kv_pages=batch * (context // PAGE),
+                         max_running=batch, step_tokens=T, prefix_cache=False)
+            ms_prefill = time_prefill(llm.steps, T, 2, vocab)
+            ms_decode, _ = time_decode_device(llm.steps, batch, context, args.steps, args.warmup, vocab)
+            llm.steps.check_status()
+            models.append({"model": f"{arch} at the {SHAPES[name][0]} layer sizes, {layers} layers",
+                           "prefill_2048_tok_s": round(T / ms_prefill * 1e3, 1), "prefill_ms": round(ms_prefill, 3),
+                           "decode_b8_ctx2048_tok_s": round(batch / ms_decode * 1e3, 1), "decode_ms_per_step": round(ms_decode, 4),
+                           "weight_gb": round(llm.model.weight_bytes() / 1e9, 3)})
+            del llm
+            torch.cuda.empty_cache()
+    table = kidarax_kernel_table(2048, 8192, 32, 64, 8, T, pk)
+    print(json.dumps({"metric": "Kidarax beside Nipadra, Pinorax and Llama at equal layer sizes (random bf16 weights)", "impl": "ours", "n_gpus": 1,
+                      "dtype": "bf16", "steps": args.steps, "warmup": args.warmup, "peaks": pk["source"],
+                      "peak_gb_s": pk["hbm_gbs"], "peak_tflops": pk["bf16_tflops"], "models": models, "kernels": table}))
+    return 0
+
+
 def run_scenario(args):
     """Two workloads through the entry point, beside the default run: ``mixed`` (32 requests with
     prompts of 128 to 4096 random ids and 256 generated tokens each, admitted together, prompts cut
@@ -1667,7 +1912,7 @@ def main():
     ap.add_argument("--shape", choices=sorted(SHAPES), default="1b", help="layer sizes (the default is the baseline's third configuration)")
     ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16",
                     help="precision of a --scenario run (float32: the requests run alone must give identical tokens)")
-    ap.add_argument("--scenario", choices=["mixed", "prefix", "sizes", "nipadra", "gekupel", "pinorax", "fovezen", "mimolix"], default="",
+    ap.add_argument("--scenario", choices=["mixed", "prefix", "sizes", "nipadra", "gekupel", "pinorax", "fovezen", "mimolix", "kidarax"], default="",
                     help="a workload through the scheduler (mixed, prefix) or decode steps at a grid of sizes, instead of the default run")
     args = ap.parse_args()
     if args.impl == "reference":
@@ -1682,6 +1927,8 @@ def main():
         return run_nipadra(args)
     if args.scenario == "gekupel":
         return run_gekupel(args)
+    if args.scenario == "kidarax":
+        return run_kidarax(args)
     if args.scenario == "mimolix":
         return run_mimolix(args)
     if args.scenario == "fovezen":

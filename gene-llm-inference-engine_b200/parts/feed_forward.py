@@ -231,35 +231,36 @@ class RoutedExpertsFeedForward:
         sorted_rows = ctx.scratch("route_sorted_rows", (tiles * tm,), torch.int32, capacity=most_tiles * tm)
         tile_group = ctx.scratch("route_tile_group", (tiles,), torch.int32, capacity=most_tiles)
         n_tiles = ctx.scratch("route_n_tiles", (1,), torch.int32, capacity=1)
-        self._route(ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles)
+        gate = self._gate(ctx, T)
+        self._route(ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles, gate)
         hidden = ctx.scratch("expert_hidden", (T * top, I), torch.float32, capacity=max(most, T) * top)
         kernels.expert_product(xn, top, self.w_first, hidden, sorted_rows, tile_group, n_tiles,
                                scales=weights if self.weigh_input else None, **self._first_form())
         part = ctx.scratch("expert_out", (T * top, D), torch.float32, capacity=max(most, T) * top)
         kernels.expert_product(hidden, 1, self.w_down, part, sorted_rows, tile_group, n_tiles)
-        self._combine(ctx, xn, part, weights, x)
+        self._combine(ctx, xn, part, weights, gate, x)
 
-    def _route(self, ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles, **tiles) -> None:
-        """The step's (token, choice) pairs and their weights, bucketed by expert."""
+    def _gate(self, ctx, T: int):
+        """Where the shared expert's gate of every token goes (None without one)."""
+        return None if self.shared_gate is None else ctx.scratch("shared_gate", (T,), torch.float32)
+
+    def _route(self, ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles, gate, **tiles) -> None:
+        """The step's (token, choice) pairs and their weights, bucketed by expert, and the shared expert's gate."""
         if self.routing == "table":
             kernels.route_table(ctx.tokens, ctx.feedback, self.table, self.experts, ids, weights, sorted_rows, tile_group, n_tiles,
                                 **tiles)
         else:
-            gate = {}
-            if self.shared_gate is not None:
-                gate = {"gate_w": self.shared_gate, "gate_out": ctx.scratch("shared_gate", (xn.shape[0],), torch.float32)}
             kernels.route(xn, self.router, self.correction, self.top, ids, weights, sorted_rows, tile_group, n_tiles,
-                          scores=self.scores, renormalise=self.renormalise, factor=self.router_scale, **gate, **tiles)
+                          scores=self.scores, renormalise=self.renormalise, factor=self.router_scale, gate_w=self.shared_gate, gate_out=gate, **tiles)
 
-    def _combine(self, ctx, xn, part, weights, x, pair_row=None) -> None:
+    def _combine(self, ctx, xn, part, weights, gate, x, pair_row=None) -> None:
         """The experts' outputs, and the shared one's, into x."""
-        more = {}
-        if self.shared_gate is not None:
+        out = None
+        if gate is not None:
             out = ctx.scratch("shared_out", tuple(x.shape), torch.float32)
             self.shared.forward(ctx, xn, out, accumulate=False)
-            more = {"more": out, "more_gate": ctx.scratch("shared_gate", (xn.shape[0],), torch.float32)}
-        kernels.route_combine(part, None if self.weigh_input else weights, x, pair_row=pair_row, top=self.top, **more)
-        if self.shared is not None and self.shared_gate is None:
+        kernels.route_combine(part, None if self.weigh_input else weights, x, pair_row=pair_row, top=self.top, more=out, more_gate=gate)
+        if self.shared is not None and gate is None:
             self.shared.forward(ctx, xn, x)
 
     def _first_form(self) -> dict:
@@ -277,11 +278,12 @@ class RoutedExpertsFeedForward:
         tile_group = ctx.scratch("route_tile_group_tc", (tiles,), torch.int32, capacity=most_tiles)
         pair_row = ctx.scratch("route_pair_row", (T * top,), torch.int32, capacity=most * top)
         n_tiles = ctx.scratch("route_n_tiles", (1,), torch.int32, capacity=1)
-        self._route(ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles, tile_rows=tm, pair_row=pair_row)
+        gate = self._gate(ctx, T)
+        self._route(ctx, xn, ids, weights, sorted_rows, tile_group, n_tiles, gate, tile_rows=tm, pair_row=pair_row)
         rows = ctx.scratch("expert_rows", (tiles * tm, D), self.dtype, capacity=most_tiles * tm)
         kernels.gather_rows(xn, top, sorted_rows, n_tiles, tm, rows, scales=weights if self.weigh_input else None)
         hidden = ctx.scratch("expert_hidden_tc", (tiles * tm, I), self.dtype, capacity=most_tiles * tm)
         kernels.expert_product_tc(rows, self.w_first, hidden, tile_group, n_tiles, **self._first_form())
         part = ctx.scratch("expert_out_tc", (tiles * tm, D), torch.float32, capacity=most_tiles * tm)
         kernels.expert_product_tc(hidden, self.w_down, part, tile_group, n_tiles)
-        self._combine(ctx, xn, part, weights, x, pair_row)
+        self._combine(ctx, xn, part, weights, gate, x, pair_row)
