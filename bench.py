@@ -1585,7 +1585,9 @@ def kidarax_kernel_table(width, ff, heads, head_dim, kv_heads, T, pk):
             def attention_work(per_tile):
                 if n == 1:
                     return rows_dec, work[:0], T
-                return rows_dec[:0], torch.tensor([(t, min(per_tile, n - t), 0) for t in range(0, n, per_tile)], **i32), 0
+                if per_tile not in Ctx.kept:          # made once; the tiles that see most keys first, as the engine orders them
+                    Ctx.kept[per_tile] = torch.tensor([(t, min(per_tile, n - t), 0) for t in range(0, n, per_tile)][::-1], **i32)
+                return rows_dec[:0], Ctx.kept[per_tile], 0
         for name, like, ep in ((f"attention_rows, a gate per value, where other sizes run ({what})", "attention_rows", {"gate": ap, "gate_offset": C}),
                                (f"attention_rows without a gate, Gekupel ({what})", "", {})):
             add(name, like, lambda: K.attention_rows_of_step(Ctx, q, kc, vc, att, tables, heads, kv_heads, head_dim, head_dim, 0.1, None, None, None, None, **ep),

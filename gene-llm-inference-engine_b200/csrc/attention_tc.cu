@@ -526,9 +526,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                 tmem_ld32(tmem_o + lane_addr + c * 32, ov);
                 tmem_ld_wait();
                 if (row_valid) {
-                    if (gz) {
+                    if (gz) {           // (16-byte pieces: the lanes' rows lie far apart)
 #pragma unroll
-                        for (int e = 0; e < 32; ++e) ov[e] = __float_as_uint(__uint_as_float(ov[e]) * sigmoid_f(gz[c * 32 + e]));
+                        for (int e = 0; e < 32; e += 4) {
+                            const float4 z = *reinterpret_cast<const float4*>(gz + c * 32 + e);
+                            ov[e] = __float_as_uint(__uint_as_float(ov[e]) * sigmoid_f(z.x));
+                            ov[e + 1] = __float_as_uint(__uint_as_float(ov[e + 1]) * sigmoid_f(z.y));
+                            ov[e + 2] = __float_as_uint(__uint_as_float(ov[e + 2]) * sigmoid_f(z.z));
+                            ov[e + 3] = __float_as_uint(__uint_as_float(ov[e + 3]) * sigmoid_f(z.w));
+                        }
                     }
 #pragma unroll
                     for (int q4 = 0; q4 < 4; ++q4) {
@@ -605,6 +611,8 @@ static int gi_attention_prefill_tc_impl(const void* q, const void* k_cache, cons
                                        float softcap, void* stream) {
     if (n_work == 0) return 0;
     const AttEpilogue ep{sink, gate, gate_ld, gate_off, gate_dims, out_scale};
+    GI_REQUIRE(gate_dims == 0 || (gate_ld % 4 == 0 && gate_off % 4 == 0 && reinterpret_cast<uintptr_t>(gate) % 16 == 0),
+               "attention_prefill_tc: the rows of a gate with a value per output must lie on 16 bytes");
     GI_REQUIRE(gi_attention_prefill_tc_supported(hd, H, Hkv, page_size), "attention_prefill_tc: shape not supported");
     GI_REQUIRE(status != nullptr, "attention_prefill_tc: a status word is required");
     GI_REQUIRE(n_work <= 65535, "attention_prefill_tc: %d work items exceed the grid limit 65535", n_work);

@@ -379,9 +379,10 @@ head_product64_kernel(const GroupedArgs p) {
 
 // ------------------------------------------------------------------------------------------------ routing
 constexpr int kRouteMaxExperts = 1024;
+constexpr int kRouteThreads = 256;
 
 template <typename TX>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kRouteThreads)
 route_kernel(const TX* __restrict__ x, int D, const float* __restrict__ w, const float* __restrict__ correction, int E, int top,
              int softmax, int renormalise, float factor, int* __restrict__ ids, float* __restrict__ weights,
              const float* __restrict__ gate_w, float* __restrict__ gate_out) {
@@ -389,12 +390,20 @@ route_kernel(const TX* __restrict__ x, int D, const float* __restrict__ w, const
     extern __shared__ float s_x[];                 // [D]
     __shared__ float s_score[kRouteMaxExperts], s_choice[kRouteMaxExperts];
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int d = threadIdx.x; d < D; d += 128) s_x[d] = to_float(x[static_cast<size_t>(t) * D + d]);
+    for (int d = threadIdx.x; d < D; d += kRouteThreads) s_x[d] = to_float(x[static_cast<size_t>(t) * D + d]);
     __syncthreads();
-    for (int e = warp; e < E + (gate_w ? 1 : 0); e += 4) {
+    for (int e = warp; e < E + (gate_w ? 1 : 0); e += kRouteThreads / 32) {
         const float* row = e < E ? w + static_cast<size_t>(e) * D : gate_w;
         float z = 0.f;
-        for (int d = lane; d < D; d += 32) z = fmaf(row[d], s_x[d], z);
+        int d = lane;
+        for (; d + 7 * 32 < D; d += 8 * 32) {            // eight loads in flight, one chain of multiply-adds
+            float v[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] = row[d + 32 * i];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) z = fmaf(v[i], s_x[d + 32 * i], z);
+        }
+        for (; d < D; d += 32) z = fmaf(row[d], s_x[d], z);
         z = warp_sum(z);
         if (e == E) {
             if (lane == 0) gate_out[t] = sigmoid_f(z);
@@ -665,10 +674,10 @@ static int gi_route_impl(const void* x, int x_dtype, int T, int D, const float* 
     const size_t smem = static_cast<size_t>(D) * 4;
     if (x_dtype == kF32) {
         if (smem > 40 * 1024) cudaFuncSetAttribute(route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-        launch_kernel((route_kernel<float>), dim3(T), dim3(128), smem, st, static_cast<const float*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights, gate_w, gate_out);
+        launch_kernel((route_kernel<float>), dim3(T), dim3(kRouteThreads), smem, st, static_cast<const float*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights, gate_w, gate_out);
     } else if (x_dtype == kBF16) {
         if (smem > 40 * 1024) cudaFuncSetAttribute(route_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-        launch_kernel((route_kernel<__nv_bfloat16>), dim3(T), dim3(128), smem, st, static_cast<const __nv_bfloat16*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights, gate_w, gate_out);
+        launch_kernel((route_kernel<__nv_bfloat16>), dim3(T), dim3(kRouteThreads), smem, st, static_cast<const __nv_bfloat16*>(x), D, w, correction, E, top, softmax, renormalise, factor, ids, weights, gate_w, gate_out);
     } else {
         GI_REQUIRE(false, "route: unsupported dtype code %d", x_dtype);
     }
